@@ -36,7 +36,7 @@
 extern "C" {
 #endif
 
-#define B2_ABI_VERSION 5
+#define B2_ABI_VERSION 6
 
 #if defined(__GNUC__)
 #define B2_API __attribute__((visibility("default")))
@@ -530,12 +530,15 @@ B2_API int b2_chunk_attention(void* out, const void* q, const void* k_cache, con
 /* b2_chunk_attention with every mask and epilogue parameter: a sliding window that keeps the sequence's first tokens
  * (position i sees j <= i with i - j < window or j < keep_first; window = 0: none), the sink's logit per query head
  * (sink_logits [H] fp32, or NULL: sink_logit for all), a sigmoid gate per (token, head) on the output (gate rows of the
- * activation type with gate_stride elements between tokens, or NULL). */
+ * activation type with gate_stride elements between tokens, or NULL), the kind of a key's weight, and output rows
+ * [H * dv] with out_stride elements between tokens.  B2_WEIGHT_SIGMOID takes head_bias [H] fp32 (or NULL: 0) and no sink. */
+#define B2_WEIGHT_SOFTMAX 0       /* exp(s_j) / (sink + sum exp(s)) */
+#define B2_WEIGHT_SIGMOID 1       /* sigmoid(s_j + head_bias[h]), not normalised over the keys */
 B2_API int b2_masked_attention(void* out, const void* q, const void* k_cache, const void* v_cache, int act_dtype,
                                const int32_t* block_tables, int max_nb, const int32_t* cu_q, const int32_t* ctx_start,
                                int n_seq, int T, int H, int G, int dk, int dv, int bs, float scale, int chunk, int window,
-                               int keep_first, float sink, float sink_logit, const float* sink_logits, const void* gate,
-                               int64_t gate_stride, void* stream);
+                               int keep_first, float sink, float sink_logit, const float* sink_logits, int weight_kind,
+                               const float* head_bias, const void* gate, int64_t gate_stride, int64_t out_stride, void* stream);
 /* rows [q (H*dk) | k (G*dk)] or [q | k | v (G*dv)]: the first rot_dims entries of every q and k head turn by the token's
  * position (pairs (i, i + rot_dims/2), or (2i, 2i+1) when interleaved; cos_sin fp32 [max_pos, rot_dims] = cos | sin
  * halves), q -> q_out [T, H, dk], rotated k -> K pool; the V pool gets v, or with v_from_k the k heads BEFORE the rotation. */
@@ -543,6 +546,12 @@ B2_API int b2_qk_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, 
                             int v_from_k, int rot_dims, int interleaved, const int32_t* positions, const float* cos_sin,
                             int max_pos, const int64_t* slots, int bs, void* q_out, void* k_cache, void* v_cache,
                             void* stream);
+/* the same after an RMS norm over all of q (H*dk numbers, weight q_w) and over all of k (G*dk, weight k_w); both weights NULL:
+ * no norm */
+B2_API int b2_qk_norm_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, int T, int H, int G, int dk, int dv,
+                                 int v_from_k, const float* q_w, const float* k_w, float eps, int rot_dims, int interleaved,
+                                 const int32_t* positions, const float* cos_sin, int max_pos, const int64_t* slots, int bs,
+                                 void* q_out, void* k_cache, void* v_cache, void* stream);
 B2_API int b2_moe_tile_rows(void);
 B2_API int b2_moe_capacity(int n, int E);
 #define B2_ROUTE_TOPK_SOFTMAX 0   /* top-k of logits + bias, weights = softmax over the chosen logits */
@@ -585,6 +594,13 @@ B2_API int b2_glu_and_mul(void* out, int64_t out_stride, const void* gate_up, in
                           int glu, float alpha, float limit, void* stream);
 B2_API int b2_gate_mul(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* gate, int64_t gate_stride,
                        int act_dtype, int T, int I, int kind, float scale, void* stream);
+/* the input row of the one output projection of a layer whose mixer and feed-forward run side by side:
+ * out[t, :n_mix] = x[t, :] * sigmoid(gate[t, :]) for t < mix_rows (gate NULL: x as it is; the columns of the other rows are not
+ * touched), out[t, n_mix + i] = act(up[t, i]) for i < n_ff.  B2_FF_XIELU: a z^2 + z/2 above zero, b (e^z - 1 - z) + z/2 below. */
+#define B2_FF_XIELU    4
+B2_API int b2_parallel_join(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* gate,
+                            int64_t gate_stride, int mix_rows, int n_mix, const void* up, int64_t up_stride, int n_ff, int ff_act,
+                            float act_a, float act_b, int act_dtype, int T, void* stream);
 B2_API int b2_softcap(void* z, int64_t stride, int act_dtype, int T, int V, float cap, void* stream);
 /* group_norm.cu: sinusoidal-position embedding, RMS norm in groups with a per-channel scale on the sublayer output and a
  * token shift (blend with the previous token's normalised row, kept per sequence in fp32 state slots) on the read-out */
@@ -606,24 +622,27 @@ B2_API int b2_latent_prep(const void* proj, int64_t proj_stride, int act_dtype, 
                           float eps, const int32_t* positions, const float* cos_sin, int max_pos, const int64_t* slots, int bs,
                           void* qa, void* cache, void* stream);
 /* b2_latent_prep with the query heads (rows q, from column q_off) and the down-projection (rows kv, from column dkv_off) in
- * two buffers */
+ * two buffers, and the rotated pairs (2i, 2i+1) (interleaved) or (i, i + rot_dims/2) */
 B2_API int b2_latent_prep_rows(const void* q, int64_t q_stride, const void* kv, int64_t kv_stride, int act_dtype, int T, int H,
-                               int dn, int dr, int rot_dims, int R, int q_off, int dkv_off, const float* norm_w, float eps,
-                               const int32_t* positions, const float* cos_sin, int max_pos, const int64_t* slots, int bs,
-                               void* qa, void* cache, void* stream);
+                               int dn, int dr, int rot_dims, int interleaved, int R, int q_off, int dkv_off,
+                               const float* norm_w, float eps, const int32_t* positions, const float* cos_sin, int max_pos,
+                               const int64_t* slots, int bs, void* qa, void* cache, void* stream);
+/* sink_logits [H] fp32 (or NULL): exp(sink_logits[h]) joins head h's softmax denominator */
 B2_API int b2_latent_attention(void* out, const void* qa, const void* cache, int act_dtype, const int32_t* block_tables,
                                int max_nb, const int32_t* cu_q, const int32_t* ctx_start, int n_seq, int T, int H, int R,
-                               int dr, int bs, float scale, int window /* 0: causal */, const void* gate /* or NULL */,
-                               int64_t gate_stride, float* workspace /* or NULL */, int64_t workspace_floats, void* stream);
+                               int dr, int bs, float scale, int window /* 0: causal */, const float* sink_logits,
+                               const void* gate /* or NULL */, int64_t gate_stride, float* workspace /* or NULL */, int64_t workspace_floats, void* stream);
 /* long prompt portions: the latent rows a portion can see, gathered to one buffer; attention over per-head keys and values
- * rebuilt from it (key = [kn[g, h, :dn] | kt[g, :dr]], query = [qn[t, h, :dn] | qr[t, h, :dr]]), sliding window, gate */
+ * rebuilt from it (key = [kn[g, h, :dn] | kt[g, :dr]], query = [qn[t, h, :dn] | qr[t, h, :dr]]), sliding window, sink, gate per
+ * head or (gate_channels) per output channel, output rows [H * dv] out_stride elements apart */
 B2_API int b2_latent_gather(void* out, const void* cache, const int32_t* block_tables, int max_nb, const int32_t* cu_k,
                             const int32_t* k_lo, int n_seq, int N, int bs, int Dc, void* stream);
 B2_API int b2_window_attention(void* out, const void* qn, int64_t qn_row, int qn_head, const void* qr, int64_t qr_row,
                                int qr_head, const void* kn, const void* kt, int64_t kt_row, const void* v,
                                const int32_t* cu_q, const int32_t* ctx_start, const int32_t* cu_k, const int32_t* k_lo,
-                               int n_seq, int T, int H, int dn, int dr, int dv, float scale, int window, const void* gate,
-                               int64_t gate_stride, void* stream);
+                               int n_seq, int T, int H, int dn, int dr, int dv, float scale, int window,
+                               const float* sink_logits, const void* gate, int64_t gate_stride, int gate_channels,
+                               int64_t out_stride, void* stream);
 B2_API int64_t b2_latent_attention_workspace(int act_dtype, int T, int n_seq, int H, int R, int dr, int bs, int window,
                                              int max_nb);
 

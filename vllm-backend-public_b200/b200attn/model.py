@@ -406,11 +406,12 @@ class LlamaModel:
 
 
 def _register_families() -> None:
-    from . import gatolix, kofadra, sanarax, tonilix
+    from . import gapidra, gatolix, kofadra, sanarax, tonilix
     ARCHITECTURES[kofadra.ARCHITECTURE] = kofadra.config_from_dir
     ARCHITECTURES[gatolix.ARCHITECTURE] = gatolix.config_from_dir
     ARCHITECTURES[tonilix.ARCHITECTURE] = tonilix.config_from_dir
     ARCHITECTURES[sanarax.ARCHITECTURE] = sanarax.config_from_dir
+    ARCHITECTURES[gapidra.ARCHITECTURE] = gapidra.config_from_dir
 
 
 _register_families()

@@ -643,8 +643,8 @@ def sample(logits: torch.Tensor, temperature: Optional[torch.Tensor] = None, see
 from dataclasses import dataclass  # noqa: E402
 
 from ._lib import (ACT_BF16, ACT_F32, DECAY_CHANNEL_SIGMOID_POW, DECAY_CHANNEL_SOFTPLUS,  # noqa: E402,F401
-                   DECAY_HEAD_CONST, DECAY_HEAD_SOFTPLUS, FF_RELU_SQ, GATE_SIGMOID, GATE_SILU, GLU_CLAMPED, GLU_GELU_TANH, GLU_SILU, NORM_LAYER,
-                   NORM_RMS, ROUTE_SIGMOID_GROUPED, ROUTE_SOFTMAX_ALL, ROUTE_TOPK_SOFTMAX)
+                   DECAY_HEAD_CONST, DECAY_HEAD_SOFTPLUS, FF_RELU_SQ, FF_XIELU, GATE_SIGMOID, GATE_SILU, GLU_CLAMPED, GLU_GELU_TANH, GLU_SILU, NORM_LAYER,
+                   NORM_RMS, ROUTE_SIGMOID_GROUPED, ROUTE_SOFTMAX_ALL, ROUTE_TOPK_SOFTMAX, WEIGHT_SIGMOID, WEIGHT_SOFTMAX)
 
 
 def _act(t: torch.Tensor, name: str) -> int:
@@ -667,6 +667,13 @@ def _mat(t: torch.Tensor, name: str):
     if t.dim() != 2 or (t.shape[1] > 1 and t.stride(1) != 1):
         raise ValueError(f"{name} must be [rows, cols] with a contiguous last axis")
     return t.shape[0], t.shape[1], (t.stride(0) if t.shape[0] > 1 else t.shape[1])
+
+
+def _out_rows(out: torch.Tensor, T: int, cols: int, dtype: torch.dtype) -> int:
+    """Row stride of an output buffer whose rows hold `cols` values one after the other, [T, cols] or [T, H, cols / H]."""
+    if out.dtype != dtype or out.shape[0] != T or out.numel() != T * cols or (T and not out[0].is_contiguous()):
+        raise ValueError(f"out must be {T} rows of {cols} values of the inputs' dtype")
+    return out.stride(0) if T > 1 else cols
 
 
 @dataclass
@@ -825,14 +832,17 @@ def qknorm_cache(qkv: torch.Tensor, H: int, G: int, dk: int, dv: int, q_w: Optio
 
 def chunk_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: SeqBatch, scale: float,
                     chunk: int = 0, sink: float = 0.0, sink_logit: float = 0.0, window: int = 0, keep_first: int = 0,
-                    sink_logits: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sink_logits: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                    weight_kind: int = WEIGHT_SOFTMAX, head_bias: Optional[torch.Tensor] = None,
+                    out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of q [T, H, dk] over the paged pools.  Row at position p sees positions j <= p with
     j // chunk == p // chunk (chunk = 0: all j <= p) and, with a window > 0, p - j < window or j < keep_first; the
     denominator carries sink * exp(sink_logit), or sink * exp(sink_logits[h]) with one fp32 logit per query head; with
     gate [T, H] (q's dtype, a column slice of a wider row is fine) head h's output is multiplied by sigmoid(gate[t, h]).
-    Returns [T, H, dv] of q's dtype.  b2_masked_attention."""
+    weight_kind WEIGHT_SIGMOID: a visible key weighs sigmoid(score + head_bias[h]) (fp32 [H] or None), not normalised; no sink.
+    Returns [T, H, dv] of q's dtype, or `out`: rows [T, >= H * dv] (a column range of a wider buffer).  b2_masked_attention."""
     lib = _lib.load()
-    dev = _need_cuda(q=q, k_cache=k_cache, v_cache=v_cache, sink_logits=sink_logits, gate=gate)
+    dev = _need_cuda(q=q, k_cache=k_cache, v_cache=v_cache, sink_logits=sink_logits, gate=gate, head_bias=head_bias, out=out)
     T, H, dk = q.shape
     nb, G, bs, dv = v_cache.shape
     if not q.is_contiguous() or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype or tuple(k_cache.shape) != (nb, G, bs, dk):
@@ -847,22 +857,29 @@ def chunk_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         if gate.dtype != q.dtype or gate.dim() != 2 or tuple(gate.shape) != (T, H) or (H > 1 and gate.stride(1) != 1):
             raise ValueError("gate must be [T, H] of q's dtype with a contiguous last axis")
         gs = gate.stride(0) if T > 1 else H
-    out = torch.empty(T, H, dv, dtype=q.dtype, device=dev)
+    _f32(head_bias, "head_bias", (H,))
+    if out is None:
+        out = torch.empty(T, H, dv, dtype=q.dtype, device=dev)
+    os_ = _out_rows(out, T, H * dv, q.dtype)
     _lib.check(lib.b2_masked_attention(_ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), _act(q, "q"), _ptr(bt), bt.shape[1],
                                        _ptr(batch.cu_q), _ptr(batch.ctx_start), batch.n_seq, T, H, G, dk, dv, bs,
                                        float(scale), int(chunk), int(window), int(keep_first), float(sink), float(sink_logit),
-                                       _ptr(sink_logits), _ptr(gate), gs, _stream(dev)))
+                                       _ptr(sink_logits), int(weight_kind), _ptr(head_bias), _ptr(gate), gs, os_, _stream(dev)))
     return out
 
 
 def qk_rope_cache(qkv: torch.Tensor, H: int, G: int, dk: int, dv: int, positions: torch.Tensor, cos_sin: Optional[torch.Tensor],
                   rot_dims: int, slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, interleaved: bool = False,
-                  v_from_k: bool = False) -> torch.Tensor:
+                  v_from_k: bool = False, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None,
+                  eps: float = 1e-6) -> torch.Tensor:
     """Rows qkv [T, >= H*dk + G*dk (+ G*dv)] = q | k (| v), biases already added: the first rot_dims entries of every q and k
     head turn by the token's position (pairs (i, i + rot_dims/2), interleaved: (2i, 2i + 1); cos_sin from rotary_table),
     rotated k goes to k_cache [nb, G, bs, dk] and v -- with v_from_k the k heads as projected, before the rotation -- to
-    v_cache [nb, G, bs, dv] at slots[t] (< 0 skips).  Returns the rotated q [T, H, dk].  b2_qk_rope_cache."""
+    v_cache [nb, G, bs, dv] at slots[t] (< 0 skips).  q_norm [H*dk] / k_norm [G*dk] (fp32, both or none): all of q and all of k
+    are RMS-normed as one row each before that.  Returns the rotated q [T, H, dk].  b2_qk_norm_rope_cache."""
     lib = _lib.load()
+    _f32(q_norm, "q_norm", (H * dk,)), _f32(k_norm, "k_norm", (G * dk,))
+    _need_cuda(q_norm=q_norm, k_norm=k_norm)
     dev = _need_cuda(qkv=qkv, slots=slots, k_cache=k_cache, v_cache=v_cache, positions=positions, cos_sin=cos_sin)
     T, P, ps = _mat(qkv, "qkv")
     if P < H * dk + G * dk + (0 if v_from_k else G * dv):
@@ -879,9 +896,10 @@ def qk_rope_cache(qkv: torch.Tensor, H: int, G: int, dk: int, dv: int, positions
                      or not cos_sin.is_contiguous()):
         raise ValueError(f"cos_sin must be contiguous fp32 [max_pos, {rot_dims}]")
     q = torch.empty(T, H, dk, dtype=qkv.dtype, device=dev)
-    _lib.check(lib.b2_qk_rope_cache(_ptr(qkv), ps, _act(qkv, "qkv"), T, H, G, dk, dv, int(v_from_k), int(rot_dims),
-                                    int(interleaved), _ptr(positions), _ptr(cos_sin), cos_sin.shape[0] if rot_dims else 1,
-                                    _ptr(slots), bs, _ptr(q), _ptr(k_cache), _ptr(v_cache), _stream(dev)))
+    _lib.check(lib.b2_qk_norm_rope_cache(_ptr(qkv), ps, _act(qkv, "qkv"), T, H, G, dk, dv, int(v_from_k), _ptr(q_norm), _ptr(k_norm),
+                                         float(eps), int(rot_dims), int(interleaved), _ptr(positions), _ptr(cos_sin),
+                                         cos_sin.shape[0] if rot_dims else 1, _ptr(slots), bs, _ptr(q), _ptr(k_cache),
+                                         _ptr(v_cache), _stream(dev)))
     return q
 
 
@@ -1208,6 +1226,36 @@ def gate_mul(x: torch.Tensor, gate: torch.Tensor, kind: int = GATE_SIGMOID, scal
     return out
 
 
+def parallel_join(out: torch.Tensor, mix: Optional[torch.Tensor], gate: Optional[torch.Tensor], n_mix: int,
+                  up: Optional[torch.Tensor], ff_act: int = FF_RELU_SQ, act_a: float = 0.0, act_b: float = 0.0) -> torch.Tensor:
+    """The input rows [T, n_mix + n_ff] of the one output projection of a layer whose mixer and feed-forward run side by side:
+    columns [0, n_mix) of the first mix.shape[0] rows become mix * sigmoid(gate) (gate None: mix; mix None: no row is touched),
+    columns [n_mix, ..) act(up).  ff_act FF_XIELU: act_a z^2 + z/2 above zero, act_b (e^z - 1 - z) + z/2 below; FF_RELU_SQ:
+    max(z, 0)^2.  b2_parallel_join."""
+    lib = _lib.load()
+    dev = _need_cuda(out=out, mix=mix, gate=gate, up=up)
+    T, C, os_ = _mat(out, "out")
+    n_ff, us = 0, 0
+    if up is not None:
+        Tu, n_ff, us = _mat(up, "up")
+        if Tu != T or up.dtype != out.dtype:
+            raise ValueError("up must be [T, n_ff] of out's dtype")
+    if C != n_mix + n_ff:
+        raise ValueError(f"out must be [T, {n_mix} + {n_ff}]")
+    rows, xs, gs = 0, 0, 0
+    if mix is not None:
+        rows, cm, xs = _mat(mix, "mix")
+        if rows > T or cm != n_mix or mix.dtype != out.dtype:
+            raise ValueError("mix must be [at most T, n_mix] of out's dtype")
+        if gate is not None:
+            Tg, cg, gs = _mat(gate, "gate")
+            if (Tg, cg) != (rows, n_mix) or gate.dtype != out.dtype:
+                raise ValueError("gate must have mix's shape and dtype")
+    _lib.check(lib.b2_parallel_join(_ptr(out), os_, _ptr(mix), xs, _ptr(gate) if mix is not None else None, gs, rows, n_mix, _ptr(up),
+                                    us, n_ff, int(ff_act), float(act_a), float(act_b), _act(out, "out"), T, _stream(dev)))
+    return out
+
+
 # ----------------------------------------------------------------------------------------------------------------------
 # csrc/post_norm.cu, csrc/latent_attention.cu
 # ----------------------------------------------------------------------------------------------------------------------
@@ -1288,7 +1336,7 @@ def softcap_(z: torch.Tensor, cap: float) -> torch.Tensor:
 
 
 def rotary_table(max_pos: int, dims: int, base: float, scaling: Optional[dict], device) -> torch.Tensor:
-    """fp32 [max_pos, dims] = cos | sin halves per position for the interleaved pairing (2i, 2i + 1), angles in fp64.
+    """fp32 [max_pos, dims] = cos | sin halves per position (column i: pair i of either pair layout), angles in fp64.
     scaling {factor, original, fast, slow} (YaRN): pairs that complete more than `fast` turns within `original` positions
     keep their frequency, pairs below `slow` turns are slowed by `factor`, a linear ramp over the pair index between the
     two; cos and sin carry the magnitude 0.1 ln(factor) + 1."""
@@ -1313,9 +1361,10 @@ def rotary_table(max_pos: int, dims: int, base: float, scaling: Optional[dict], 
 def latent_prep(proj: torch.Tensor, H: int, dn: int, dr: int, rot_dims: int, R: int, q_off: int, dkv_off: int,
                 norm_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor, cos_sin: torch.Tensor,
                 slots: Optional[torch.Tensor], cache: Optional[torch.Tensor], qa: Optional[torch.Tensor] = None,
-                kv: Optional[torch.Tensor] = None) -> torch.Tensor:
+                kv: Optional[torch.Tensor] = None, interleaved: bool = True) -> torch.Tensor:
     """Rows proj [T, ...] hold the query heads [dn | dr] from column q_off and, when dkv_off >= 0, the down-projection
-    [R | dr] from column dkv_off -- of proj, or of kv [T, ...] when the two come out of different products.  Writes the rotated dr part of every query head to qa[t, h, R:], and (dkv_off >= 0) the
+    [R | dr] from column dkv_off -- of proj, or of kv [T, ...] when the two come out of different products.  Writes the dr part of every query head, its first
+    rot_dims entries rotated (pairs (2i, 2i + 1), or (i, i + rot_dims/2) when not interleaved), to qa[t, h, R:], and (dkv_off >= 0) the
     RMS-normed latent and the rotated shared key part to cache [nb, bs, R + dr] at slots[t] (< 0 skips).  Returns qa
     [T, H, R + dr] of proj's dtype, whose first R columns per head are left for the absorbed query.  b2_latent_prep."""
     lib = _lib.load()
@@ -1342,19 +1391,21 @@ def latent_prep(proj: torch.Tensor, H: int, dn: int, dr: int, rot_dims: int, R: 
         qa = torch.empty(T, H, R + dr, dtype=proj.dtype, device=dev)
     elif tuple(qa.shape) != (T, H, R + dr) or qa.dtype != proj.dtype or not qa.is_contiguous():
         raise ValueError("qa must be contiguous [T, H, R + dr] of proj's dtype")
-    _lib.check(lib.b2_latent_prep_rows(_ptr(proj), ps, _ptr(kv), ks, _act(proj, "proj"), T, H, dn, dr, rot_dims, R, q_off, dkv_off,
-                                       _ptr(norm_w), float(eps), _ptr(positions), _ptr(cos_sin), cos_sin.shape[0], _ptr(slots),
+    _lib.check(lib.b2_latent_prep_rows(_ptr(proj), ps, _ptr(kv), ks, _act(proj, "proj"), T, H, dn, dr, rot_dims, int(interleaved), R, q_off,
+                                       dkv_off, _ptr(norm_w), float(eps), _ptr(positions), _ptr(cos_sin), cos_sin.shape[0], _ptr(slots),
                                        bs, _ptr(qa), _ptr(cache) if dkv_off >= 0 else None, _stream(dev)))
     return qa
 
 
 def latent_attention(qa: torch.Tensor, cache: torch.Tensor, batch: SeqBatch, R: int, scale: float, window: int = 0,
-                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, sink_logits: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Absorbed queries qa [T, H, R + dr] against the latent pool cache [nb, bs, R + dr]: the row at position p sees
     positions j <= p (window > 0: and p - j < window); returns sigmoid(gate[t, h]) * sum_j p_j cache[j, :R] as
-    [T, H, R] of qa's dtype.  gate [T, H] may be a column slice of a wider row.  b2_latent_attention."""
+    [T, H, R] of qa's dtype.  gate [T, H] may be a column slice of a wider row.  sink_logits fp32 [H]: exp(sink_logits[h]) joins
+    the denominator of head h.  b2_latent_attention."""
     lib = _lib.load()
-    dev = _need_cuda(qa=qa, cache=cache, gate=gate)
+    dev = _need_cuda(qa=qa, cache=cache, gate=gate, sink_logits=sink_logits)
+    _f32(sink_logits, "sink_logits", (qa.shape[1],))
     T, H, Dc = qa.shape
     if not qa.is_contiguous() or cache.dtype != qa.dtype or cache.dim() != 3 or cache.shape[2] != Dc or not cache.is_contiguous():
         raise ValueError("qa must be contiguous and cache [nb, bs, R + dr] of its dtype")
@@ -1373,7 +1424,7 @@ def latent_attention(qa: torch.Tensor, cache: torch.Tensor, batch: SeqBatch, R: 
     ws = torch.empty(nws, dtype=torch.float32, device=dev) if nws else None
     _lib.check(lib.b2_latent_attention(_ptr(out), _ptr(qa), _ptr(cache), _act(qa, "qa"), _ptr(bt), bt.shape[1], _ptr(batch.cu_q),
                                        _ptr(batch.ctx_start), batch.n_seq, T, H, R, Dc - R, cache.shape[1], float(scale),
-                                       int(window), _ptr(gate), gs, _ptr(ws), nws, _stream(dev)))
+                                       int(window), _ptr(sink_logits), _ptr(gate), gs, _ptr(ws), nws, _stream(dev)))
     return out
 
 
@@ -1418,14 +1469,16 @@ def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, cu_k: torch.T
 
 def window_attention(qn: torch.Tensor, qr: torch.Tensor, kn: torch.Tensor, kt: torch.Tensor, v: torch.Tensor, cu_q: torch.Tensor,
                      ctx_start: torch.Tensor, cu_k: torch.Tensor, k_lo: torch.Tensor, n_seq: int, scale: float, window: int = 0,
-                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, sink_logits: Optional[torch.Tensor] = None,
+                     out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Sliding-window attention of prompt portions over keys and values held per head in gathered buffers.
     qn [T, H, dn], qr [T, H, dr]: the two parts of the queries (views with a contiguous last axis); kn [N, H, dn], kt [N, dr]
     (shared by the heads; may be a column slice), v [N, H, dv] over the gathered rows (see latent_gather).  The row at
-    position p sees positions max(0, p - window + 1) .. p (window 0: 0 .. p).  Returns sigmoid(gate[t, h]) * softmax(..) v as
-    bf16 [T, H, dv].  b2_window_attention."""
+    position p sees positions max(0, p - window + 1) .. p (window 0: 0 .. p); sink_logits fp32 [H]: exp(sink_logits[h]) joins the
+    denominator.  Returns sigmoid(gate) * softmax(..) v as bf16 [T, H, dv], gate [T, H] or one column per channel [T, H * dv]; or
+    `out`: rows of H * dv values (a column range of a wider buffer).  b2_window_attention."""
     lib = _lib.load()
-    dev = _need_cuda(qn=qn, qr=qr, kn=kn, kt=kt, v=v, gate=gate)
+    dev = _need_cuda(qn=qn, qr=qr, kn=kn, kt=kt, v=v, gate=gate, sink_logits=sink_logits, out=out)
     T, H, dn = qn.shape
     dr, dv, N = qr.shape[2], v.shape[2], kn.shape[0]
     if tuple(qr.shape) != (T, H, dr) or tuple(kn.shape) != (N, H, dn) or tuple(kt.shape) != (N, dr) or tuple(v.shape) != (N, H, dv):
@@ -1435,14 +1488,18 @@ def window_attention(qn: torch.Tensor, qr: torch.Tensor, kn: torch.Tensor, kt: t
             raise ValueError(f"{name} must be bf16 with a contiguous last axis")
     if not kn.is_contiguous() or not v.is_contiguous():
         raise ValueError("kn and v must be contiguous")
-    gs = 0
+    _f32(sink_logits, "sink_logits", (H,))
+    gs, channels = 0, False
     if gate is not None:
-        if gate.dtype != torch.bfloat16 or tuple(gate.shape) != (T, H) or (H > 1 and gate.stride(1) != 1):
-            raise ValueError("gate must be bf16 [T, H] with a contiguous last axis")
-        gs = gate.stride(0) if T > 1 else H
-    out = torch.empty(T, H, dv, dtype=torch.bfloat16, device=dev)
+        if gate.dtype != torch.bfloat16 or tuple(gate.shape) not in ((T, H), (T, H * dv)) or (gate.shape[1] > 1 and gate.stride(1) != 1):
+            raise ValueError("gate must be bf16 [T, H] or [T, H * dv] with a contiguous last axis")
+        channels = gate.shape[1] != H
+        gs = gate.stride(0) if T > 1 else gate.shape[1]
+    if out is None:
+        out = torch.empty(T, H, dv, dtype=torch.bfloat16, device=dev)
+    os_ = _out_rows(out, T, H * dv, torch.bfloat16)
     _lib.check(lib.b2_window_attention(_ptr(out), _ptr(qn), qn.stride(0), qn.stride(1), _ptr(qr), qr.stride(0), qr.stride(1),
                                        _ptr(kn), _ptr(kt), kt.stride(0), _ptr(v), _ptr(cu_q), _ptr(ctx_start), _ptr(cu_k),
-                                       _ptr(k_lo), n_seq, T, H, dn, dr, dv, float(scale), int(window), _ptr(gate), gs,
-                                       _stream(dev)))
+                                       _ptr(k_lo), n_seq, T, H, dn, dr, dv, float(scale), int(window), _ptr(sink_logits),
+                                       _ptr(gate), gs, int(channels), os_, _stream(dev)))
     return out

@@ -53,6 +53,10 @@ __device__ __forceinline__ float relu_sq_f(float z) {
     z = fmaxf(z, 0.f);
     return z * z;
 }
+// quadratic above zero, exponential below, plus half the identity: a z^2 + z/2, b (e^z - 1 - z) + z/2
+__device__ __forceinline__ float xielu_f(float z, float a, float b) {
+    return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (expm1f(z) - z));
+}
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // four consecutive elements of an activation row (8 or 16 bytes, aligned)

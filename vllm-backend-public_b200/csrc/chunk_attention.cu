@@ -1,5 +1,5 @@
-// chunk_attention.cu -- softmax attention without a rotation over a paged cache, with three parameters that other
-// designs can set independently:
+// chunk_attention.cu -- attention over a paged cache of keys and values per kv head, with parameters that designs set
+// independently of each other:
 //   * per-head RMS norm of queries and keys (a plain weight of size dk shared by the heads),
 //   * a block-local causal mask: position i sees j <= i with floor(j / chunk) == floor(i / chunk), blocks counted from
 //     position 0 of the sequence (chunk = 0: plain causal),
@@ -8,7 +8,9 @@
 //     query head (sink_logits [H], not scaled),
 //   * a sliding window that keeps the first tokens: position i sees j <= i with i - j < window or j < keep_first
 //     (window = 0: no window).  A query then reads the kept keys and its window's keys and nothing between them,
-//   * a sigmoid gate per (token, head) on the head's output.
+//   * a sigmoid gate per (token, head) on the head's output,
+//   * the weight of a visible key: its share of the softmax, or (B2_WEIGHT_SIGMOID) sigmoid(score + head_bias[h]), a number
+//     of its own that no other key changes -- no maximum, no denominator, and a sink has no meaning.
 // Key size dk and value size dv are independent; K and V live in separate paged pools
 //   k_cache [num_blocks, G, bs, dk],  v_cache [num_blocks, G, bs, dv]      (activation type).
 //
@@ -21,6 +23,9 @@
 //                        token's position (pairs (i, i + rot_dims/2) or (2i, 2i + 1); fp32 table [max_pos, rot_dims] =
 //                        cos | sin halves), q to q_out, rotated k to the K pool; the V pool receives v, or, for designs
 //                        whose values ARE the keys, the k heads as projected (before the rotation).
+//   b2_qk_norm_rope_cache  rows [q | k | v]: all of q (H * dk numbers) and all of k (G * dk) are RMS-normed as one row each,
+//                        before the split into heads (fp32 weights of those sizes), then rotated and written as above; the
+//                        numbers stay in fp32 between the norm and the rotation.
 //   b2_chunk_attention   per (token, head) one warp: scores of 32 keys at a time (a lane per key), online softmax in fp32
 //                        seeded with the sink, P.V with a lane per value column.  With the mask a query touches at most
 //                        `chunk` keys wherever it stands, so prompt chunks and decode rows run the same kernel; a decode
@@ -52,14 +57,34 @@ __device__ __forceinline__ bool key_visible(int i, int j, int lo_i, int window, 
     return j <= i && j >= lo_i && (window <= 0 || i - j < window || j < keep_first);
 }
 
-// Rows [q | k] (+ [v]): partial rotation of the q and k heads, K (rotated) and V pool writes; see the file comment.
-template <typename T>
+// 1 / rms of all H * dk numbers of q and of all G * dk of k, which lie one after the other at `src` (block-wide)
+template <typename T, int W>
+__device__ __forceinline__ void qk_row_scales(const T* src, int nq, int nk, float eps, float* red, float& inv_q, float& inv_k) {
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x * W; i < nq + nk; i += blockDim.x * W) {
+        float v[4] = {0.f, 0.f, 0.f, 0.f}, ss = 0.f;
+        if (W == 4) b2::ld4(src + i, v); else v[0] = b2::ld(src + i);
+#pragma unroll
+        for (int c = 0; c < W; ++c) ss = fmaf(v[c], v[c], ss);
+        if (i < nq) sq += ss; else sk += ss;
+    }
+    inv_q = rsqrtf(b2::block_sum(sq, red) / (float)nq + eps);
+    inv_k = rsqrtf(b2::block_sum(sk, red) / (float)nk + eps);
+}
+
+// Rows [q | k] (+ [v]): partial rotation of the q and k heads, K (rotated) and V pool writes; see the file comment.  NORM:
+// q and k are first normed over their whole rows.
+template <typename T, bool NORM>
 __global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, int G, int dk, int dv, bool v_from_k,
                                      int rot_dims, bool interleaved, const int32_t* __restrict__ positions,
                                      const float* __restrict__ cos_sin, int max_pos, const int64_t* __restrict__ slots, int bs,
+                                     const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                                      T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache) {
+    __shared__ float red[33];
     const int row = blockIdx.x;
     const T* src = qkv + (size_t)row * qkv_stride;
+    float inv_q = 1.f, inv_k = 1.f;
+    if (NORM) qk_row_scales<T, 1>(src, H * dk, G * dk, eps, red, inv_q, inv_k);
     int pos = positions[row];
     pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
     const float* cs = cos_sin + (size_t)pos * rot_dims;
@@ -72,13 +97,16 @@ __global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stri
         const int hd = idx / dk, i = idx % dk;
         if (hd >= H && slot < 0) continue;
         const T* v = src + (size_t)hd * dk;
+        const float* w = NORM ? (hd < H ? q_w + (size_t)hd * dk : k_w + (size_t)(hd - H) * dk) : nullptr;
+        const float inv = hd < H ? inv_q : inv_k;
         float x = b2::ld(v + i);
+        if (NORM) x *= inv * w[i];
         if (i < rot_dims) {
             int pr, partner;
             bool second;
             if (interleaved) { pr = i >> 1; partner = i ^ 1; second = i & 1; }
             else { second = i >= half; pr = second ? i - half : i; partner = second ? i - half : i + half; }
-            const float c = cs[pr], sn = cs[half + pr], other = b2::ld(v + partner);
+            const float c = cs[pr], sn = cs[half + pr], other = b2::ld(v + partner) * (NORM ? inv * w[partner] : 1.f);
             x = second ? fmaf(x, c, other * sn) : fmaf(x, c, -other * sn);
         }
         T* dst = hd < H ? q_out + ((size_t)row * H + hd) * dk : k_cache + (((size_t)blk * G + (hd - H)) * bs + off) * dk;
@@ -94,14 +122,17 @@ __global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stri
 
 // The same with four entries per access (8 or 16 bytes): every size a multiple of four, the rotated entries a multiple of
 // eight in the (i, i + rot_dims/2) layout so that a group of four and its partners never straddle the halves.
-template <typename T>
+template <typename T, bool NORM>
 __global__ void __launch_bounds__(256)
 qk_rope_cache_vec_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, int G, int dk, int dv, bool v_from_k, int rot_dims,
                          bool interleaved, const int32_t* __restrict__ positions, const float* __restrict__ cos_sin, int max_pos,
-                         const int64_t* __restrict__ slots, int bs, T* __restrict__ q_out, T* __restrict__ k_cache,
-                         T* __restrict__ v_cache) {
+                         const int64_t* __restrict__ slots, int bs, const float* __restrict__ q_w, const float* __restrict__ k_w,
+                         float eps, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache) {
+    __shared__ float red[33];
     const int row = blockIdx.x;
     const T* src = qkv + (size_t)row * qkv_stride;
+    float inv_q = 1.f, inv_k = 1.f;
+    if (NORM) qk_row_scales<T, 4>(src, H * dk, G * dk, eps, red, inv_q, inv_k);
     int pos = positions[row];
     pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
     const float* cs = cos_sin + (size_t)pos * rot_dims;
@@ -113,8 +144,14 @@ qk_rope_cache_vec_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, i
     for (int idx = threadIdx.x; idx < nqk; idx += blockDim.x) {
         const int hd = idx / per, i = (idx % per) * 4;
         const T* v = src + (size_t)hd * dk;
+        const float* w = NORM ? (hd < H ? q_w + (size_t)hd * dk : k_w + (size_t)(hd - H) * dk) : nullptr;
+        const float inv = hd < H ? inv_q : inv_k;
         float x[4];
         b2::ld4(v + i, x);
+        if (NORM) {
+#pragma unroll
+            for (int c = 0; c < 4; ++c) x[c] *= inv * w[i + c];
+        }
         if (i < rot_dims) {
             if (interleaved) {
 #pragma unroll
@@ -126,10 +163,12 @@ qk_rope_cache_vec_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, i
             } else {
                 const bool second = i >= half;
                 const int pr = second ? i - half : i;
+                const int pi = second ? i - half : i + half;
                 float y[4];
-                b2::ld4(v + (second ? i - half : i + half), y);
+                b2::ld4(v + pi, y);
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
+                    if (NORM) y[c] *= inv * w[pi + c];
                     const float co = cs[pr + c], si = cs[half + pr + c];
                     x[c] = second ? fmaf(x[c], co, y[c] * si) : fmaf(x[c], co, -y[c] * si);
                 }
@@ -196,14 +235,17 @@ __global__ void qknorm_cache_kernel(const T* __restrict__ qkv, int64_t qkv_strid
     }
 }
 
-template <typename T>
+// sigmoid of a score that is already in the exponent of 2
+__device__ __forceinline__ float sigmoid2_f(float x2) { return __fdividef(1.f, 1.f + exp2f(-x2)); }
+
+template <typename T, bool SIG>
 __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                                        const int32_t* __restrict__ block_tables, int max_nb,
                                        const int32_t* __restrict__ cu_q, const int32_t* __restrict__ ctx_start, int n_seq,
                                        int rows, int H, int G, int dk, int dv, int bs, float scale, int chunk, int window,
                                        int keep_first, float sink, float sink_logit, const float* __restrict__ sink_logits,
-                                       const T* __restrict__ gate, int64_t gate_stride, int skip_rows_from,
-                                       T* __restrict__ out) {
+                                       const float* __restrict__ head_bias, const T* __restrict__ gate, int64_t gate_stride,
+                                       int skip_rows_from, T* __restrict__ out, int64_t out_stride) {
     extern __shared__ float q_sm[];                  // [warps, dk]
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const int item = blockIdx.x * (blockDim.x >> 5) + wid;       // (row, head)
@@ -211,7 +253,7 @@ __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restr
     const int row = item / H, hh = item % H;
     const int seq = b2::seq_of_row(cu_q, n_seq, row);
     const int ctx = ctx_start[seq];
-    T* dst = out + (size_t)item * dv;
+    T* dst = out + (size_t)row * out_stride + (size_t)hh * dv;
     if (skip_rows_from > 0 && ctx >= 0 && cu_q[seq + 1] - cu_q[seq] >= skip_rows_from) return;    // the tile kernel's
     if (ctx < 0) {
         for (int i = lane; i < dv; i += 32) b2::st(dst + i, 0.f);
@@ -226,6 +268,7 @@ __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restr
     __syncwarp();
     const int32_t* bt = block_tables + (size_t)seq * max_nb;
     float m = sink > 0.f ? (sink_logits ? sink_logits[hh] : sink_logit) : -INFINITY, l = sink;      // the sink seeds the running maximum and denominator
+    const float bias = SIG && head_bias ? head_bias[hh] : 0.f;
     float acc[kMaxDvPerLane];
 #pragma unroll
     for (int c = 0; c < kMaxDvPerLane; ++c) acc[c] = 0.f;
@@ -242,13 +285,18 @@ __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restr
             for (int i = 0; i < dk; ++i) d = fmaf(qs[i], b2::ld(kr + i), d);
             s = d;
         }
-        const float m_new = fmaxf(m, b2::warp_max(s));
-        const float corr = m == -INFINITY ? 0.f : __expf(m - m_new);
-        const float p = in ? __expf(s - m_new) : 0.f;
-        l = l * corr + b2::warp_sum(p);
-        m = m_new;
+        float p;
+        if (SIG) {
+            p = in ? b2::sigmoid_f(s + bias) : 0.f;
+        } else {
+            const float m_new = fmaxf(m, b2::warp_max(s));
+            const float corr = m == -INFINITY ? 0.f : __expf(m - m_new);
+            p = in ? __expf(s - m_new) : 0.f;
+            l = l * corr + b2::warp_sum(p);
+            m = m_new;
 #pragma unroll
-        for (int c = 0; c < kMaxDvPerLane; ++c) acc[c] *= corr;
+            for (int c = 0; c < kMaxDvPerLane; ++c) acc[c] *= corr;
+        }
         const int nk = min(32, span.n - c0);
         for (int kk = 0; kk < nk; ++kk) {
             const float pk = __shfl_sync(0xffffffffu, p, kk);
@@ -261,7 +309,7 @@ __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restr
             }
         }
     }
-    float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = SIG ? 1.f : (l > 0.f ? 1.f / l : 0.f);
     if (gate) inv *= b2::sigmoid_f(b2::ld(gate + (size_t)row * gate_stride + hh));
 #pragma unroll
     for (int c = 0; c < kMaxDvPerLane; ++c) {
@@ -282,13 +330,15 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(b2::smem_u32(dst)), "l"(src) : "memory");
 }
 
+template <bool SIG>
 __global__ void __launch_bounds__(128)
 chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                              const __nv_bfloat16* __restrict__ v_cache, const int32_t* __restrict__ block_tables, int max_nb,
                              const int32_t* __restrict__ cu_q, const int32_t* __restrict__ ctx_start, int n_seq, int H, int G,
                              int dk, int dv, int bs, float scale, int chunk, int window, int keep_first, float sink,
-                             float sink_logit, const float* __restrict__ sink_logits, const __nv_bfloat16* __restrict__ gate,
-                             int64_t gate_stride, int skip_rows_from, __nv_bfloat16* __restrict__ out) {
+                             float sink_logit, const float* __restrict__ sink_logits, const float* __restrict__ head_bias,
+                             const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, int skip_rows_from,
+                             __nv_bfloat16* __restrict__ out, int64_t out_stride) {
     // q [QH][dk] | per warp: m [QH], l [QH], acc [QH][dv] | per warp: K tile [32][dk + 8], V tile [32][dv] (bf16)
     extern __shared__ __align__(16) float grp_sm[];
     const int row = blockIdx.x, g = blockIdx.y;
@@ -298,7 +348,8 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
     const int QHall = H / G;
     if (skip_rows_from > 0 && ctx >= 0 && cu_q[seq + 1] - cu_q[seq] >= skip_rows_from) return;    // the tile kernel's
     if (ctx < 0) {
-        for (int i = tid; i < QHall * dv; i += 128) out[((size_t)row * H + (size_t)g * QHall) * dv + i] = __float2bfloat16_rn(0.f);
+        for (int i = tid; i < QHall * dv; i += 128)
+            out[(size_t)row * out_stride + (size_t)g * QHall * dv + i] = __float2bfloat16_rn(0.f);
         return;
     }
     const int pos = ctx + row - cu_q[seq];
@@ -321,6 +372,7 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
         for (int h = 0; h < kGroupMaxHeads; ++h) {
             m[h] = (w == 0 && sink > 0.f) ? (sink_logits ? sink_logits[g * QHall + h0 + min(h, QH - 1)] : sink_logit) : -INFINITY;
             l[h] = w == 0 ? sink : 0.f;
+            if (SIG) m[h] = head_bias ? head_bias[g * QHall + h0 + min(h, QH - 1)] : 0.f;      // holds the head's bias instead
 #pragma unroll
             for (int c = 0; c < kGroupMaxPairs; ++c) acc[h][c][0] = acc[h][c][1] = 0.f;
         }
@@ -371,7 +423,9 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
 #pragma unroll
             for (int h = 0; h < kGroupMaxHeads; ++h) {
                 pr[h] = 0.f;
-                if (h < QH) {
+                if (SIG) {
+                    if (h < QH && valid) pr[h] = b2::sigmoid_f(sc[h] + m[h]);
+                } else if (h < QH) {
                     const float x = valid ? sc[h] : -INFINITY;
                     const float mn = fmaxf(m[h], b2::warp_max(x));          // finite: the tile has at least one key
                     const float corr = m[h] == -INFINITY ? 0.f : __expf(m[h] - mn);
@@ -432,10 +486,14 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
         __syncthreads();
         for (int i = tid; i < QH * dv; i += 128) {
             const int h = i / dv, col = i % dv;
-            float M = -INFINITY;
-            for (int x = 0; x < 4; ++x) M = fmaxf(M, part[((size_t)x * kGroupMaxHeads + h) * (2 + dv)]);
-            float L = 0.f, O = 0.f;
-            if (M > -INFINITY) {
+            float M = -INFINITY, L = 0.f, O = 0.f;
+            if (SIG) {
+                L = 1.f;
+                for (int x = 0; x < 4; ++x) O += part[((size_t)x * kGroupMaxHeads + h) * (2 + dv) + 2 + col];
+            } else {
+                for (int x = 0; x < 4; ++x) M = fmaxf(M, part[((size_t)x * kGroupMaxHeads + h) * (2 + dv)]);
+            }
+            if (!SIG && M > -INFINITY) {
                 for (int x = 0; x < 4; ++x) {
                     const float* px = part + ((size_t)x * kGroupMaxHeads + h) * (2 + dv);
                     const float f = px[0] == -INFINITY ? 0.f : __expf(px[0] - M);
@@ -445,7 +503,7 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
             }
             float res = L > 0.f ? O / L : 0.f;
             if (gate) res *= b2::sigmoid_f(__bfloat162float(gate[(size_t)row * gate_stride + (size_t)g * QHall + h0 + h]));
-            out[((size_t)row * H + (size_t)g * QHall + h0 + h) * dv + col] = __float2bfloat16_rn(res);
+            out[(size_t)row * out_stride + ((size_t)g * QHall + h0 + h) * dv + col] = __float2bfloat16_rn(res);
         }
     }
 }
@@ -459,14 +517,15 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
 // kTileMinRows rows (decode rows) are left to the warp kernel above.
 constexpr int kTQ = 64, kTK = 64, kTileMinRows = 16;
 
-template <int DKT, int DVT>
+template <int DKT, int DVT, bool SIG>
 __global__ void __launch_bounds__(128)
 chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                             const __nv_bfloat16* __restrict__ v_cache, const int32_t* __restrict__ block_tables, int max_nb,
                             const int32_t* __restrict__ cu_q, const int32_t* __restrict__ ctx_start, int n_seq, int H, int G,
                             int bs, float scale_log2, int chunk, int window, int keep_first, float sink,
-                            float sink_logit_log2, const float* __restrict__ sink_logits,
-                            const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, __nv_bfloat16* __restrict__ out) {
+                            float sink_logit_log2, const float* __restrict__ sink_logits, const float* __restrict__ head_bias,
+                            const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, __nv_bfloat16* __restrict__ out,
+                            int64_t out_stride) {
     constexpr int DK = 16 * DKT, DV = 16 * DVT, LDK = DK + 8, LDV = DV + 8;
     extern __shared__ __align__(16) unsigned char tile_smem[];
     __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(tile_smem);      // [64][LDK]
@@ -512,6 +571,7 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     if (sink_logits) sink_logit_log2 = sink_logits[hh] * 1.4426950408889634f;
     float m0 = sink > 0.f ? sink_logit_log2 : -INFINITY, m1 = m0;
     float l0 = tq == 0 ? sink : 0.f, l1 = l0;                               // partial sums per lane; the sink counted once
+    const float bias_log2 = SIG && head_bias ? head_bias[hh] * 1.4426950408889634f : 0.f;
     float o[2 * DVT][4];
 #pragma unroll
     for (int n = 0; n < 2 * DVT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -552,45 +612,57 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                 b2::mma_bf16_16816(sc[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
             }
         }
-        float mx0 = -INFINITY, mx1 = -INFINITY;
+        if (SIG) {                                                          // every weight by itself: nothing to rescale
 #pragma unroll
-        for (int n = 0; n < 8; ++n) {
+            for (int n = 0; n < 8; ++n) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
-                const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
-                sc[n][e] = ok ? sc[n][e] * scale_log2 : -INFINITY;
+                for (int e = 0; e < 4; ++e) {
+                    const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
+                    const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
+                    sc[n][e] = ok ? sigmoid2_f(fmaf(sc[n][e], scale_log2, bias_log2)) : 0.f;
+                }
             }
-            mx0 = fmaxf(mx0, fmaxf(sc[n][0], sc[n][1]));
-            mx1 = fmaxf(mx1, fmaxf(sc[n][2], sc[n][3]));
-        }
-        mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-        mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-        mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-        mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-        const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-        const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
-        const float c0 = exp2f(m0 - mu0), c1 = exp2f(m1 - mu1);             // exp2(-inf) = 0: nothing accumulated yet
-        m0 = mn0;
-        m1 = mn1;
-        float s0 = 0.f, s1 = 0.f;
+        } else {
+            float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
-        for (int n = 0; n < 8; ++n) {
-            sc[n][0] = exp2f(sc[n][0] - mu0);
-            sc[n][1] = exp2f(sc[n][1] - mu0);
-            sc[n][2] = exp2f(sc[n][2] - mu1);
-            sc[n][3] = exp2f(sc[n][3] - mu1);
-            s0 += sc[n][0] + sc[n][1];
-            s1 += sc[n][2] + sc[n][3];
-        }
-        l0 = l0 * c0 + s0;
-        l1 = l1 * c1 + s1;
+            for (int n = 0; n < 8; ++n) {
 #pragma unroll
-        for (int n = 0; n < 2 * DVT; ++n) {
-            o[n][0] *= c0;
-            o[n][1] *= c0;
-            o[n][2] *= c1;
-            o[n][3] *= c1;
+                for (int e = 0; e < 4; ++e) {
+                    const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
+                    const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
+                    sc[n][e] = ok ? sc[n][e] * scale_log2 : -INFINITY;
+                }
+                mx0 = fmaxf(mx0, fmaxf(sc[n][0], sc[n][1]));
+                mx1 = fmaxf(mx1, fmaxf(sc[n][2], sc[n][3]));
+            }
+            mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+            mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+            mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+            mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+            const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
+            const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
+            const float c0 = exp2f(m0 - mu0), c1 = exp2f(m1 - mu1);             // exp2(-inf) = 0: nothing accumulated yet
+            m0 = mn0;
+            m1 = mn1;
+            float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+            for (int n = 0; n < 8; ++n) {
+                sc[n][0] = exp2f(sc[n][0] - mu0);
+                sc[n][1] = exp2f(sc[n][1] - mu0);
+                sc[n][2] = exp2f(sc[n][2] - mu1);
+                sc[n][3] = exp2f(sc[n][3] - mu1);
+                s0 += sc[n][0] + sc[n][1];
+                s1 += sc[n][2] + sc[n][3];
+            }
+            l0 = l0 * c0 + s0;
+            l1 = l1 * c1 + s1;
+#pragma unroll
+            for (int n = 0; n < 2 * DVT; ++n) {
+                o[n][0] *= c0;
+                o[n][1] *= c0;
+                o[n][2] *= c1;
+                o[n][3] *= c1;
+            }
         }
 #pragma unroll
         for (int ks = 0; ks < 4; ++ks) {
@@ -611,7 +683,7 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-    float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+    float inv0 = SIG ? 1.f : (l0 > 0.f ? 1.f / l0 : 0.f), inv1 = SIG ? 1.f : (l1 > 0.f ? 1.f / l1 : 0.f);
     const int ra = w * 16 + gq, rb = ra + 8;
     if (gate) {
         if (ra < rows) inv0 *= b2::sigmoid_f(__bfloat162float(gate[(size_t)(r0 + ra) * gate_stride + hh]));
@@ -621,27 +693,28 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     for (int n = 0; n < 2 * DVT; ++n) {
         const int col = n * 8 + 2 * tq;
         if (ra < rows)
-            *reinterpret_cast<uint32_t*>(out + ((size_t)(r0 + ra) * H + hh) * DV + col) = b2::pack_bf16x2(o[n][0] * inv0, o[n][1] * inv0);
+            *reinterpret_cast<uint32_t*>(out + (size_t)(r0 + ra) * out_stride + hh * DV + col) = b2::pack_bf16x2(o[n][0] * inv0, o[n][1] * inv0);
         if (rb < rows)
-            *reinterpret_cast<uint32_t*>(out + ((size_t)(r0 + rb) * H + hh) * DV + col) = b2::pack_bf16x2(o[n][2] * inv1, o[n][3] * inv1);
+            *reinterpret_cast<uint32_t*>(out + (size_t)(r0 + rb) * out_stride + hh * DV + col) = b2::pack_bf16x2(o[n][2] * inv1, o[n][3] * inv1);
     }
 }
 
-template <int DKT, int DVT>
+template <int DKT, int DVT, bool SIG>
 int launch_tile(const void* q, const void* k_cache, const void* v_cache, const int32_t* block_tables, int max_nb,
                 const int32_t* cu_q, const int32_t* ctx_start, int n_seq, int T, int H, int G, int bs, float scale, int chunk,
-                int window, int keep_first, float sink, float sink_logit, const float* sink_logits, const void* gate,
-                int64_t gate_stride, void* out, cudaStream_t st) {
+                int window, int keep_first, float sink, float sink_logit, const float* sink_logits, const float* head_bias,
+                const void* gate, int64_t gate_stride, void* out, int64_t out_stride, cudaStream_t st) {
     constexpr int DK = 16 * DKT, DV = 16 * DVT;
     const size_t smem = (size_t)(kTQ * (DK + 8) + kTK * (DK + 8) + kTK * (DV + 8)) * sizeof(__nv_bfloat16);
-    auto kern = chunk_attention_tile_kernel<DKT, DVT>;
+    auto kern = chunk_attention_tile_kernel<DKT, DVT, SIG>;
     if (smem > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const int tiles = (T + kTQ - 1) / kTQ + n_seq;          // upper bound on sum(ceil(len / 64)); spare CTAs leave at once
     kern<<<dim3(tiles, H), 128, smem, st>>>(static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
                                            static_cast<const __nv_bfloat16*>(v_cache), block_tables, max_nb, cu_q, ctx_start,
                                            n_seq, H, G, bs, scale * 1.4426950408889634f, chunk, window, keep_first, sink,
-                                           sink_logit * 1.4426950408889634f, sink_logits,
-                                           static_cast<const __nv_bfloat16*>(gate), gate_stride, static_cast<__nv_bfloat16*>(out));
+                                           sink_logit * 1.4426950408889634f, sink_logits, head_bias,
+                                           static_cast<const __nv_bfloat16*>(gate), gate_stride, static_cast<__nv_bfloat16*>(out),
+                                           out_stride);
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }
@@ -685,11 +758,20 @@ extern "C" int b2_qk_rope_cache(const void* qkv, int64_t qkv_stride, int act_dty
                                 int v_from_k, int rot_dims, int interleaved, const int32_t* positions, const float* cos_sin,
                                 int max_pos, const int64_t* slots, int bs, void* q_out, void* k_cache, void* v_cache,
                                 void* stream) {
+    return b2_qk_norm_rope_cache(qkv, qkv_stride, act_dtype, T, H, G, dk, dv, v_from_k, nullptr, nullptr, 0.f, rot_dims, interleaved,
+                                 positions, cos_sin, max_pos, slots, bs, q_out, k_cache, v_cache, stream);
+}
+
+extern "C" int b2_qk_norm_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, int T, int H, int G, int dk, int dv,
+                                     int v_from_k, const float* q_w, const float* k_w, float eps, int rot_dims, int interleaved,
+                                     const int32_t* positions, const float* cos_sin, int max_pos, const int64_t* slots, int bs,
+                                     void* q_out, void* k_cache, void* v_cache, void* stream) {
     B2_REQUIRE(T >= 0 && H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0 && bs > 0, B2_EINVAL, "qk_rope_cache: bad sizes");
     B2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk, B2_EINVAL,
                "qk_rope_cache: %d rotated entries in heads of %d", rot_dims, dk);
     B2_REQUIRE(!v_from_k || dv == dk, B2_EINVAL, "qk_rope_cache: values taken from the keys need dv == dk");
     B2_REQUIRE(rot_dims == 0 || max_pos > 0, B2_EINVAL, "qk_rope_cache: empty rotation table");
+    B2_REQUIRE(!q_w == !k_w, B2_EINVAL, "qk_rope_cache: the norm needs the weights of both q and k");
     if (T == 0) return B2_OK;
     B2_REQUIRE(qkv && slots && q_out && k_cache && v_cache && positions && (cos_sin || rot_dims == 0), B2_EINVAL,
                "qk_rope_cache: null pointer");
@@ -700,16 +782,17 @@ extern "C" int b2_qk_rope_cache(const void* qkv, int64_t qkv_stride, int act_dty
                      al(k_cache) && al(v_cache);
     const int work = (H + G) * dk / (vec ? 4 : 1);
     const int threads = work >= 256 ? 256 : (work >= 128 ? 128 : 64);
+#define B2_ROPE(KERN, NORM)                                                                                                     \
+    KERN<A, NORM><<<T, threads, 0, st>>>(static_cast<const A*>(qkv), qkv_stride, H, G, dk, dv, v_from_k != 0, rot_dims,         \
+                                         interleaved != 0, positions, cos_sin, max_pos > 0 ? max_pos : 1, slots, bs, q_w, k_w, eps, \
+                                         static_cast<A*>(q_out), static_cast<A*>(k_cache), static_cast<A*>(v_cache))
     B2_DISPATCH_ACT(act_dtype, A, {
-        if (vec)
-            qk_rope_cache_vec_kernel<A><<<T, threads, 0, st>>>(
-                static_cast<const A*>(qkv), qkv_stride, H, G, dk, dv, v_from_k != 0, rot_dims, interleaved != 0, positions, cos_sin,
-                max_pos > 0 ? max_pos : 1, slots, bs, static_cast<A*>(q_out), static_cast<A*>(k_cache), static_cast<A*>(v_cache));
-        else
-            qk_rope_cache_kernel<A><<<T, threads, 0, st>>>(
-                static_cast<const A*>(qkv), qkv_stride, H, G, dk, dv, v_from_k != 0, rot_dims, interleaved != 0, positions, cos_sin,
-                max_pos > 0 ? max_pos : 1, slots, bs, static_cast<A*>(q_out), static_cast<A*>(k_cache), static_cast<A*>(v_cache));
+        if (vec && q_w) B2_ROPE(qk_rope_cache_vec_kernel, true);
+        else if (vec) B2_ROPE(qk_rope_cache_vec_kernel, false);
+        else if (q_w) B2_ROPE(qk_rope_cache_kernel, true);
+        else B2_ROPE(qk_rope_cache_kernel, false);
     });
+#undef B2_ROPE
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }
@@ -719,17 +802,25 @@ extern "C" int b2_chunk_attention(void* out, const void* q, const void* k_cache,
                                   int n_seq, int T, int H, int G, int dk, int dv, int bs, float scale, int chunk, float sink,
                                   float sink_logit, void* stream) {
     return b2_masked_attention(out, q, k_cache, v_cache, act_dtype, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, dk, dv,
-                               bs, scale, chunk, 0, 0, sink, sink_logit, nullptr, nullptr, 0, stream);
+                               bs, scale, chunk, 0, 0, sink, sink_logit, nullptr, B2_WEIGHT_SOFTMAX, nullptr, nullptr, 0,
+                               (int64_t)H * dv, stream);
 }
 
 extern "C" int b2_masked_attention(void* out, const void* q, const void* k_cache, const void* v_cache, int act_dtype,
                                    const int32_t* block_tables, int max_nb, const int32_t* cu_q, const int32_t* ctx_start,
                                    int n_seq, int T, int H, int G, int dk, int dv, int bs, float scale, int chunk, int window,
-                                   int keep_first, float sink, float sink_logit, const float* sink_logits, const void* gate,
-                                   int64_t gate_stride, void* stream) {
+                                   int keep_first, float sink, float sink_logit, const float* sink_logits, int weight_kind,
+                                   const float* head_bias, const void* gate, int64_t gate_stride, int64_t out_stride,
+                                   void* stream) {
     B2_REQUIRE(T >= 0 && H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0 && bs > 0 && chunk >= 0 && sink >= 0.f && window >= 0 &&
                keep_first >= 0, B2_EINVAL, "masked_attention: bad sizes");
     B2_REQUIRE(!gate || gate_stride >= H, B2_EINVAL, "masked_attention: gate rows shorter than the heads");
+    B2_REQUIRE(weight_kind == B2_WEIGHT_SOFTMAX || weight_kind == B2_WEIGHT_SIGMOID, B2_EINVAL,
+               "masked_attention: unknown weight kind %d", weight_kind);
+    const bool sig = weight_kind == B2_WEIGHT_SIGMOID;
+    B2_REQUIRE(sig ? sink == 0.f : !head_bias, B2_EINVAL,
+               "masked_attention: sigmoid weights have no sink, and only they take a bias per head");
+    B2_REQUIRE(out_stride >= (int64_t)H * dv, B2_EINVAL, "masked_attention: output rows shorter than the heads");
     B2_REQUIRE(dv <= 32 * kMaxDvPerLane, B2_EUNSUPPORTED, "chunk_attention: value size %d above %d", dv, 32 * kMaxDvPerLane);
     if (T == 0 || n_seq == 0) return B2_OK;
     B2_REQUIRE(out && q && k_cache && v_cache && block_tables && cu_q && ctx_start, B2_EINVAL, "chunk_attention: null pointer");
@@ -742,13 +833,17 @@ extern "C" int b2_masked_attention(void* out, const void* q, const void* k_cache
     // kTileMinRows rows, so a batch of T rows over n_seq sequences can only hold one when T - n_seq >= kTileMinRows - 1)
     int skip_from = 0;
     if (act_dtype == B2_ACT_BF16 && T - n_seq >= kTileMinRows - 1 && dk % 32 == 0 && dv % 32 == 0 && dk <= 128 && dv <= 128 &&
-        b2_aligned16(q) && b2_aligned16(k_cache) && b2_aligned16(v_cache) && b2_aligned16(out)) {
+        b2_aligned16(q) && b2_aligned16(k_cache) && b2_aligned16(v_cache) && b2_aligned16(out) && out_stride % 8 == 0) {
         skip_from = kTileMinRows;
         int rc = B2_OK;
 #define B2_TILE(a, b)                                                                                                     \
     if (dk == 16 * a && dv == 16 * b)                                                                                     \
-        rc = launch_tile<a, b>(q, k_cache, v_cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, bs, scale, chunk, \
-                               window, keep_first, sink, sink_logit, sink_logits, gate, gate_stride, out, st);
+        rc = sig ? launch_tile<a, b, true>(q, k_cache, v_cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, bs, scale, \
+                                           chunk, window, keep_first, 0.f, 0.f, nullptr, head_bias, gate, gate_stride, out,       \
+                                           out_stride, st)                                                                        \
+                 : launch_tile<a, b, false>(q, k_cache, v_cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, bs, scale, \
+                                            chunk, window, keep_first, sink, sink_logit, sink_logits, nullptr, gate, gate_stride, \
+                                            out, out_stride, st);
         B2_TILE(2, 2) B2_TILE(2, 4) B2_TILE(2, 6) B2_TILE(2, 8) B2_TILE(4, 2) B2_TILE(4, 4) B2_TILE(4, 6) B2_TILE(4, 8)
         B2_TILE(6, 2) B2_TILE(6, 4) B2_TILE(6, 6) B2_TILE(6, 8) B2_TILE(8, 2) B2_TILE(8, 4) B2_TILE(8, 6) B2_TILE(8, 8)
 #undef B2_TILE
@@ -759,21 +854,27 @@ extern "C" int b2_masked_attention(void* out, const void* q, const void* k_cache
         const size_t gsm = (size_t)(kGroupMaxHeads * dk + 4 * kGroupMaxHeads * (2 + dv)) * sizeof(float) +
                            (size_t)4 * 32 * (dk + 8 + dv) * sizeof(__nv_bfloat16);
         if (gsm <= 160 * 1024) {
-            auto kern = chunk_attention_group_kernel;
+            auto kern = sig ? chunk_attention_group_kernel<true> : chunk_attention_group_kernel<false>;
             if (gsm > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gsm));
             kern<<<dim3(T, G), 128, gsm, st>>>(static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
                                                static_cast<const __nv_bfloat16*>(v_cache), block_tables, max_nb, cu_q, ctx_start,
                                                n_seq, H, G, dk, dv, bs, scale, chunk, window, keep_first, sink, sink_logit,
-                                               sink_logits, static_cast<const __nv_bfloat16*>(gate), gate_stride, skip_from,
-                                               static_cast<__nv_bfloat16*>(out));
+                                               sink_logits, head_bias, static_cast<const __nv_bfloat16*>(gate), gate_stride,
+                                               skip_from, static_cast<__nv_bfloat16*>(out), out_stride);
             B2_CUDA_OK(cudaGetLastError());
             return B2_OK;
         }
     }
-    B2_DISPATCH_ACT(act_dtype, A, (chunk_attention_kernel<A><<<blocks, warps * 32, smem, st>>>(
-        static_cast<const A*>(q), static_cast<const A*>(k_cache), static_cast<const A*>(v_cache), block_tables, max_nb, cu_q,
-        ctx_start, n_seq, T, H, G, dk, dv, bs, scale, chunk, window, keep_first, sink, sink_logit, sink_logits,
-        static_cast<const A*>(gate), gate_stride, skip_from, static_cast<A*>(out))));
+#define B2_WARP_ATTENTION(SIG)                                                                                                \
+    chunk_attention_kernel<A, SIG><<<blocks, warps * 32, smem, st>>>(                                                         \
+        static_cast<const A*>(q), static_cast<const A*>(k_cache), static_cast<const A*>(v_cache), block_tables, max_nb, cu_q, \
+        ctx_start, n_seq, T, H, G, dk, dv, bs, scale, chunk, window, keep_first, sink, sink_logit, sink_logits, head_bias,    \
+        static_cast<const A*>(gate), gate_stride, skip_from, static_cast<A*>(out), out_stride)
+    B2_DISPATCH_ACT(act_dtype, A, {
+        if (sig) B2_WARP_ATTENTION(true);
+        else B2_WARP_ATTENTION(false);
+    });
+#undef B2_WARP_ATTENTION
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }

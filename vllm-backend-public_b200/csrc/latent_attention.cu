@@ -7,16 +7,19 @@
 // straight against the cache rows, and the head's output is W_uv[h] applied to sum_j p_j c_j.  Every head reads the same
 // R + dr numbers per key: the op is multi-query attention with key size R + dr and value = the first R entries of the key.
 //
-//   b2_latent_prep        per token: the rotated parts of the query heads are rotated (pairs 2i, 2i+1 of the first
-//                         `rot_dims` entries; angle and magnitude from a fp32 table [max_pos, rot_dims] = cos | sin halves)
+//   b2_latent_prep        per token: the rotated parts of the query heads are rotated (pairs (2i, 2i+1) or, half layout,
+//                         (i, i + rot_dims/2) of the first `rot_dims` entries; angle and magnitude from a fp32 table
+//                         [max_pos, rot_dims] = cos | sin halves)
 //                         and written behind the absorbed part of qa; when the layer owns a down-projection its first R
 //                         outputs are RMS-normed (plain weight) into the cache row at the token's slot and the last dr,
 //                         rotated, behind them.  A layer that reads another layer's pool passes dkv_off < 0.
 //   b2_latent_prep_rows   the same with the query heads and the down-projection in rows of two different buffers (a design
-//                         whose queries come out of a second product, behind a query latent).
+//                         whose queries come out of a second product, behind a query latent) and the pair layout chosen.
 //   b2_latent_attention   o[t, h, :R] = gate[t, h] * sum_j softmax_j(s)[j] c_j over the visible keys: j <= i, and with a
 //                         window W > 0 also i - j < W.  gate = sigmoid of a per-head column of the projection rows
-//                         (gate NULL: 1).  Softmax state, scores and the accumulator are fp32.
+//                         (gate NULL: 1).  A sink adds exp(sink_logits[h]) to head h's denominator, a key without a value
+//                         (sink_logits NULL: none; not scaled, counted once also when a row's keys are split over CTAs).
+//                         Softmax state, scores and the accumulator are fp32.
 // Sequences are described like everywhere in this library: rows cu_q[i] .. cu_q[i+1]-1, ctx_start[i] cached tokens before
 // them (< 0: padding, output rows are zeroed), block_tables[i, :].
 // Every sequence of a batch has at least one row; a batch with as many rows as sequences is therefore one row each (a
@@ -27,10 +30,22 @@
 namespace {
 
 constexpr int kMaxRPerLane = 32;                     // R <= 1024 in the warp kernel
+constexpr float kLog2e = 1.4426950408889634f;
+
+// entry i < rot_dims of a part that turns: partner entry and pair index in either layout; `second`: i is the pair's second entry
+struct RotPair {
+    int pair, partner;
+    bool second;
+};
+__device__ __forceinline__ RotPair rot_pair(int i, int half, bool interleaved) {
+    if (interleaved) return {i >> 1, i ^ 1, (i & 1) != 0};
+    const bool second = i >= half;
+    return {second ? i - half : i, second ? i - half : i + half, second};
+}
 
 template <typename T>
 __global__ void latent_prep_kernel(const T* __restrict__ proj, int64_t proj_stride, const T* __restrict__ kv, int64_t kv_stride,
-                                   int H, int dn, int dr, int rot_dims, int R,
+                                   int H, int dn, int dr, int rot_dims, bool interleaved, int R,
                                    int q_off, int dkv_off, const float* __restrict__ norm_w, float eps,
                                    const int32_t* __restrict__ positions, const float* __restrict__ cos_sin, int max_pos,
                                    const int64_t* __restrict__ slots, int bs, T* __restrict__ qa, T* __restrict__ cache) {
@@ -47,10 +62,10 @@ __global__ void latent_prep_kernel(const T* __restrict__ proj, int64_t proj_stri
         const T* src = row + q_off + (size_t)hh * (dn + dr) + dn;
         float v = b2::ld(src + i);
         if (i < rot_dims) {
-            const int pr = i >> 1;
-            const float c = cs[pr], s = cs[half + pr];
-            const float other = b2::ld(src + (i ^ 1));
-            v = (i & 1) ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
+            const RotPair r = rot_pair(i, half, interleaved);
+            const float c = cs[r.pair], s = cs[half + r.pair];
+            const float other = b2::ld(src + r.partner);
+            v = r.second ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
         }
         b2::st(qa + ((size_t)t * H + hh) * Dc + R + i, v);
     }
@@ -69,19 +84,20 @@ __global__ void latent_prep_kernel(const T* __restrict__ proj, int64_t proj_stri
     for (int i = threadIdx.x; i < dr; i += blockDim.x) {
         float v = b2::ld(src + R + i);
         if (i < rot_dims) {
-            const int pr = i >> 1;
-            const float c = cs[pr], s = cs[half + pr];
-            const float other = b2::ld(src + R + (i ^ 1));
-            v = (i & 1) ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
+            const RotPair r = rot_pair(i, half, interleaved);
+            const float c = cs[r.pair], s = cs[half + r.pair];
+            const float other = b2::ld(src + R + r.partner);
+            v = r.second ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
         }
         b2::st(dst + R + i, v);
     }
 }
 
-// The same with four elements per access (8 or 16 bytes) for row layouts whose offsets are all multiples of four.
+// The same with four elements per access (8 or 16 bytes) for row layouts whose offsets are all multiples of four; in the half
+// layout rot_dims is a multiple of eight, so that a group of four and its partners never straddle the halves.
 template <typename T>
 __global__ void latent_prep_vec_kernel(const T* __restrict__ proj, int64_t proj_stride, const T* __restrict__ kv,
-                                       int64_t kv_stride, int H, int dn, int dr, int rot_dims, int R,
+                                       int64_t kv_stride, int H, int dn, int dr, int rot_dims, bool interleaved, int R,
                                        int q_off, int dkv_off, const float* __restrict__ norm_w, float eps,
                                        const int32_t* __restrict__ positions, const float* __restrict__ cos_sin, int max_pos,
                                        const int64_t* __restrict__ slots, T* __restrict__ qa, T* __restrict__ cache) {
@@ -92,22 +108,35 @@ __global__ void latent_prep_vec_kernel(const T* __restrict__ proj, int64_t proj_
     int pos = positions[t];
     pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
     const float* cs = cos_sin + (size_t)pos * rot_dims;
-    auto turn = [&](float (&v)[4], int i) {          // entries i .. i+3 of a rotated part: two pairs
+    auto turn = [&](float (&v)[4], int i, const T* part) {      // entries i .. i+3 of the rotated part at `part`
+        if (interleaved) {                           // two whole pairs
 #pragma unroll
-        for (int c = 0; c < 4; c += 2) {
-            if (i + c < rot_dims) {
-                const int pr = (i + c) >> 1;
-                const float co = cs[pr], si = cs[half + pr], u = v[c], w = v[c + 1];
-                v[c] = u * co - w * si;
-                v[c + 1] = w * co + u * si;
+            for (int c = 0; c < 4; c += 2) {
+                if (i + c < rot_dims) {
+                    const int pr = (i + c) >> 1;
+                    const float co = cs[pr], si = cs[half + pr], u = v[c], w = v[c + 1];
+                    v[c] = u * co - w * si;
+                    v[c + 1] = w * co + u * si;
+                }
+            }
+        } else if (i < rot_dims) {                   // four first or four second entries; their partners are a group too
+            const bool second = i >= half;
+            const int pr = second ? i - half : i;
+            float y[4];
+            b2::ld4(part + (second ? i - half : i + half), y);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const float co = cs[pr + c], si = cs[half + pr + c];
+                v[c] = second ? fmaf(v[c], co, y[c] * si) : fmaf(v[c], co, -y[c] * si);
             }
         }
     };
     for (int e = threadIdx.x * 4; e < H * dr; e += blockDim.x * 4) {
         const int hh = e / dr, i = e % dr;
+        const T* part = row + q_off + (size_t)hh * (dn + dr) + dn;
         float v[4];
-        b2::ld4(row + q_off + (size_t)hh * (dn + dr) + dn + i, v);
-        turn(v, i);
+        b2::ld4(part + i, v);
+        turn(v, i, part);
         b2::st4(qa + ((size_t)t * H + hh) * Dc + R + i, v);
     }
     if (dkv_off < 0) return;
@@ -132,7 +161,7 @@ __global__ void latent_prep_vec_kernel(const T* __restrict__ proj, int64_t proj_
     for (int i = threadIdx.x * 4; i < dr; i += blockDim.x * 4) {
         float v[4];
         b2::ld4(src + R + i, v);
-        turn(v, i);
+        turn(v, i, src + R);
         b2::st4(dst + R + i, v);
     }
 }
@@ -143,8 +172,8 @@ template <typename T>
 __global__ void latent_attention_kernel(const T* __restrict__ qa, const T* __restrict__ cache,
                                         const int32_t* __restrict__ block_tables, int max_nb, const int32_t* __restrict__ cu_q,
                                         const int32_t* __restrict__ ctx_start, int n_seq, int rows, int H, int R, int dr, int bs,
-                                        float scale, int window, const T* __restrict__ gate, int64_t gate_stride,
-                                        T* __restrict__ out) {
+                                        float scale, int window, const float* __restrict__ sink_logits,
+                                        const T* __restrict__ gate, int64_t gate_stride, T* __restrict__ out) {
     extern __shared__ float q_sm[];                  // [warps, R + dr]
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const int item = blockIdx.x * (blockDim.x >> 5) + wid;       // (row, head)
@@ -165,7 +194,7 @@ __global__ void latent_attention_kernel(const T* __restrict__ qa, const T* __res
     for (int i = lane; i < Dc; i += 32) qs[i] = b2::ld(qv + i) * scale;
     __syncwarp();
     const int32_t* bt = block_tables + (size_t)seq * max_nb;
-    float m = -INFINITY, l = 0.f;
+    float m = sink_logits ? sink_logits[hh] : -INFINITY, l = sink_logits ? 1.f : 0.f;     // the sink seeds maximum and denominator
     float acc[kMaxRPerLane];
 #pragma unroll
     for (int c = 0; c < kMaxRPerLane; ++c) acc[c] = 0.f;
@@ -234,8 +263,9 @@ __global__ void __launch_bounds__(256)
 latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bfloat16* __restrict__ cache,
                             const int32_t* __restrict__ block_tables, int max_nb, const int32_t* __restrict__ cu_q,
                             const int32_t* __restrict__ ctx_start, int n_seq, int H, int Hc, int dr, int bs, float scale_log2,
-                            int window, int stages, const __nv_bfloat16* __restrict__ gate, int64_t gate_stride,
-                            __nv_bfloat16* __restrict__ out, float* __restrict__ ws_o, float* __restrict__ ws_ml) {
+                            int window, int stages, const float* __restrict__ sink_logits,
+                            const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, __nv_bfloat16* __restrict__ out,
+                            float* __restrict__ ws_o, float* __restrict__ ws_ml) {
     constexpr int R = 16 * RT;
     const int Dc = R + dr, LD = Dc + 8, vecs = Dc / 8;
     extern __shared__ __align__(16) unsigned char lat_smem[];
@@ -295,6 +325,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bfl
     const int w_first = p0 + (wm * 16) / Hc, w_last = p0 + (wm * 16 + 15) / Hc;
     const int w_lo = window > 0 ? max(w_first - window + 1, 0) : 0;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    if (sink_logits && zs == 0) {                                           // the sink belongs to the first share of the keys
+        m0 = sink_logits[h0 + min(ra % Hc, nh - 1)] * kLog2e;
+        m1 = sink_logits[h0 + min(rb % Hc, nh - 1)] * kLog2e;
+        if (tq == 0) l0 = l1 = 1.f;                                         // partial sums per lane: counted once
+    }
     float o[RT][4];
 #pragma unroll
     for (int n = 0; n < RT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -456,8 +491,9 @@ __global__ void __launch_bounds__(256)
 latent_attention_decode_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bfloat16* __restrict__ cache,
                                const int32_t* __restrict__ block_tables, int max_nb, const int32_t* __restrict__ cu_q,
                                const int32_t* __restrict__ ctx_start, int H, int dr, int bs, float scale_log2, int window,
-                               const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, __nv_bfloat16* __restrict__ out,
-                               float* __restrict__ ws_o, float* __restrict__ ws_ml) {
+                               const float* __restrict__ sink_logits, const __nv_bfloat16* __restrict__ gate,
+                               int64_t gate_stride, __nv_bfloat16* __restrict__ out, float* __restrict__ ws_o,
+                               float* __restrict__ ws_ml) {
     constexpr int R = 16 * RT, CW = R / 8, NTO = CW / 8;                    // output columns / n-tiles per warp
     static_assert(CW % 16 == 0, "a warp owns whole pairs of n-tiles");
     const int Dc = R + dr, LD = Dc + 8, vecs = Dc / 8;
@@ -496,6 +532,11 @@ latent_attention_decode_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_
     }
     const int gq = lane >> 2, tq = lane & 3;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    if (sink_logits && zs == 0) {                                           // every warp keeps the same maximum, its own sums
+        m0 = sink_logits[h0 + min(gq, nh - 1)] * kLog2e;
+        m1 = sink_logits[h0 + min(gq + 8, nh - 1)] * kLog2e;
+        if (w == 0 && tq == 0) l0 = l1 = 1.f;
+    }
     float o[NTO][4];
 #pragma unroll
     for (int n = 0; n < NTO; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -641,6 +682,8 @@ latent_attention_decode_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_
 // per-head keys and values come from two library GEMMs over that buffer, and b2_window_attention runs over them:
 //   key of head h at gathered row g = [ kn[g, h, :dn] | kt[g, :dr] ]   (kt: the shared rotated part, a column slice of
 //   the gathered rows), value v[g, h, :dv]; query = [ qn[t, h, :dn] | qr[t, h, :dr] ] from two buffers as well.
+// The gate is one column per head or (gate_channels) one per output channel, and the output rows have a stride of their own
+// (they may be a column range of a wider buffer).
 // One CTA = 64 consecutive rows of one sequence x one head, four warps of 16 rows, 64-key tiles staged through shared
 // memory, mma.sync m16n8k16 with ldmatrix operands, online softmax in registers (exp2, scale folded in).  bf16; dn and dr
 // multiples of 8, dn + dr and dv multiples of 16, dv <= 128.
@@ -663,7 +706,8 @@ window_attention_kernel(const __nv_bfloat16* __restrict__ qn, int64_t qn_row, in
                         int64_t kt_row, const __nv_bfloat16* __restrict__ v, const int32_t* __restrict__ cu_q,
                         const int32_t* __restrict__ ctx_start, const int32_t* __restrict__ cu_k, const int32_t* __restrict__ k_lo,
                         int n_seq, int H, int dn, int dr, int dv, float scale_log2, int window,
-                        const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, __nv_bfloat16* __restrict__ out) {
+                        const float* __restrict__ sink_logits, const __nv_bfloat16* __restrict__ gate, int64_t gate_stride,
+                        bool gate_channels, __nv_bfloat16* __restrict__ out, int64_t out_stride) {
     const int DK = dn + dr, LDK = DK + 8, LDV = dv + 8, dkt = DK / 16, dvt = dv / 16;
     extern __shared__ __align__(16) unsigned char lat_smem[];
     __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(lat_smem);       // [64][LDK]
@@ -686,7 +730,8 @@ window_attention_kernel(const __nv_bfloat16* __restrict__ qn, int64_t qn_row, in
     const int ctx = ctx_start[seq];
     if (ctx < 0) {
         for (int idx = tid; idx < rows * (dv / 8); idx += 128)
-            *reinterpret_cast<uint4*>(out + ((size_t)(r0 + idx / (dv / 8)) * H + hh) * dv + (idx % (dv / 8)) * 8) = make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint4*>(out + (size_t)(r0 + idx / (dv / 8)) * out_stride + (size_t)hh * dv + (idx % (dv / 8)) * 8) =
+                make_uint4(0, 0, 0, 0);
         return;
     }
     const int p0 = ctx + t0, p_last = p0 + rows - 1;
@@ -709,7 +754,8 @@ window_attention_kernel(const __nv_bfloat16* __restrict__ qn, int64_t qn_row, in
     const int lo0 = window > 0 ? max(i0 - window + 1, 0) : 0, lo1 = window > 0 ? max(i1 - window + 1, 0) : 0;
     const int w_first = p0 + w * 16, w_last = w_first + 15;
     const int w_lo = window > 0 ? max(w_first - window + 1, 0) : 0;
-    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    const float seed = sink_logits ? sink_logits[hh] * kLog2e : -INFINITY;
+    float m0 = seed, m1 = seed, l0 = sink_logits && tq == 0 ? 1.f : 0.f, l1 = l0;
     float o[2 * kWMaxDVT][4];
 #pragma unroll
     for (int n = 0; n < 2 * kWMaxDVT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -819,18 +865,28 @@ window_attention_kernel(const __nv_bfloat16* __restrict__ qn, int64_t qn_row, in
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     const int ra = w * 16 + gq, rb = ra + 8;
     float f0 = l0 > 0.f ? 1.f / l0 : 0.f, f1 = l1 > 0.f ? 1.f / l1 : 0.f;
-    if (gate) {
-        if (ra < rows) f0 *= b2::sigmoid_f(__bfloat162float(gate[(size_t)(r0 + ra) * gate_stride + hh]));
-        if (rb < rows) f1 *= b2::sigmoid_f(__bfloat162float(gate[(size_t)(r0 + rb) * gate_stride + hh]));
+    const __nv_bfloat16* ga = gate ? gate + (size_t)(r0 + ra) * gate_stride : nullptr;
+    const __nv_bfloat16* gb = gate ? gate + (size_t)(r0 + rb) * gate_stride : nullptr;
+    if (gate && !gate_channels) {
+        if (ra < rows) f0 *= b2::sigmoid_f(__bfloat162float(ga[hh]));
+        if (rb < rows) f1 *= b2::sigmoid_f(__bfloat162float(gb[hh]));
     }
+    auto gated = [&](const __nv_bfloat16* g, int col, float x, float y) {
+        if (gate && gate_channels) {
+            const uint32_t z = *reinterpret_cast<const uint32_t*>(g + (size_t)hh * dv + col);
+            x *= b2::sigmoid_f(__uint_as_float(z << 16));
+            y *= b2::sigmoid_f(__uint_as_float(z & 0xffff0000u));
+        }
+        return b2::pack_bf16x2(x, y);
+    };
+    __nv_bfloat16* oa = out + (size_t)(r0 + ra) * out_stride + (size_t)hh * dv;
+    __nv_bfloat16* ob = out + (size_t)(r0 + rb) * out_stride + (size_t)hh * dv;
 #pragma unroll
     for (int n = 0; n < 2 * kWMaxDVT; ++n) {
         const int col = n * 8 + 2 * tq;
         if (col < dv) {
-            if (ra < rows)
-                *reinterpret_cast<uint32_t*>(out + ((size_t)(r0 + ra) * H + hh) * dv + col) = b2::pack_bf16x2(o[n][0] * f0, o[n][1] * f0);
-            if (rb < rows)
-                *reinterpret_cast<uint32_t*>(out + ((size_t)(r0 + rb) * H + hh) * dv + col) = b2::pack_bf16x2(o[n][2] * f1, o[n][3] * f1);
+            if (ra < rows) *reinterpret_cast<uint32_t*>(oa + col) = gated(ga, col, o[n][0] * f0, o[n][1] * f0);
+            if (rb < rows) *reinterpret_cast<uint32_t*>(ob + col) = gated(gb, col, o[n][2] * f1, o[n][3] * f1);
         }
     }
 }
@@ -891,8 +947,9 @@ inline LatentPlan latent_plan(int T, int n_seq, int H, int R, int window, int ma
 
 template <int RT>
 int launch_latent_mma(void* out, const void* qa, const void* cache, const int32_t* block_tables, int max_nb, const int32_t* cu_q,
-                      const int32_t* ctx_start, int n_seq, int T, int H, int dr, int bs, float scale, int window, const void* gate,
-                      int64_t gate_stride, bool decode, int nsplit, float* ws, cudaStream_t st) {
+                      const int32_t* ctx_start, int n_seq, int T, int H, int dr, int bs, float scale, int window,
+                      const float* sink_logits, const void* gate, int64_t gate_stride, bool decode, int nsplit, float* ws,
+                      cudaStream_t st) {
     const int Dc = 16 * RT + dr, Hc = H < kLQ ? H : kLQ, Gt = kLQ / Hc;
     const size_t tile = (size_t)kLK * (Dc + 8) * sizeof(__nv_bfloat16);
     const int stages = 3 * tile <= 227 * 1024 - 64 ? 2 : 1;                 // two key tiles in flight when they fit beside Q
@@ -910,7 +967,7 @@ int launch_latent_mma(void* out, const void* qa, const void* cache, const int32_
             if (dsm > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(dk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dsm));
             dk<<<dim3(T, (H + 15) / 16, nsplit), 256, dsm, st>>>(
                 static_cast<const __nv_bfloat16*>(qa), static_cast<const __nv_bfloat16*>(cache), block_tables, max_nb, cu_q, ctx_start,
-                H, dr, bs, scale * 1.4426950408889634f, window, static_cast<const __nv_bfloat16*>(gate), gate_stride,
+                H, dr, bs, scale * kLog2e, window, sink_logits, static_cast<const __nv_bfloat16*>(gate), gate_stride,
                 static_cast<__nv_bfloat16*>(out), ws_o, ws_ml);
             if (nsplit > 1)
                 latent_merge_kernel<<<T * H, 128, 0, st>>>(ws_o, ws_ml, nsplit, 16 * RT, H, static_cast<const __nv_bfloat16*>(gate),
@@ -921,7 +978,7 @@ int launch_latent_mma(void* out, const void* qa, const void* cache, const int32_
     }
     kern<<<dim3(tiles, (H + Hc - 1) / Hc, nsplit), 256, smem, st>>>(
         static_cast<const __nv_bfloat16*>(qa), static_cast<const __nv_bfloat16*>(cache), block_tables, max_nb, cu_q, ctx_start,
-        n_seq, H, Hc, dr, bs, scale * 1.4426950408889634f, window, stages, static_cast<const __nv_bfloat16*>(gate), gate_stride,
+        n_seq, H, Hc, dr, bs, scale * kLog2e, window, stages, sink_logits, static_cast<const __nv_bfloat16*>(gate), gate_stride,
         static_cast<__nv_bfloat16*>(out), ws_o, ws_ml);
     if (nsplit > 1)
         latent_merge_kernel<<<T * H, 128, 0, st>>>(ws_o, ws_ml, nsplit, 16 * RT, H, static_cast<const __nv_bfloat16*>(gate),
@@ -949,14 +1006,14 @@ extern "C" int b2_latent_prep(const void* proj, int64_t proj_stride, int act_dty
                               int R, int q_off, int dkv_off, const float* norm_w, float eps, const int32_t* positions,
                               const float* cos_sin, int max_pos, const int64_t* slots, int bs, void* qa, void* cache,
                               void* stream) {
-    return b2_latent_prep_rows(proj, proj_stride, proj, proj_stride, act_dtype, T, H, dn, dr, rot_dims, R, q_off, dkv_off, norm_w,
+    return b2_latent_prep_rows(proj, proj_stride, proj, proj_stride, act_dtype, T, H, dn, dr, rot_dims, 1, R, q_off, dkv_off, norm_w,
                                eps, positions, cos_sin, max_pos, slots, bs, qa, cache, stream);
 }
 
 extern "C" int b2_latent_prep_rows(const void* q, int64_t q_stride, const void* kv, int64_t kv_stride, int act_dtype, int T, int H,
-                                   int dn, int dr, int rot_dims, int R, int q_off, int dkv_off, const float* norm_w, float eps,
-                                   const int32_t* positions, const float* cos_sin, int max_pos, const int64_t* slots, int bs,
-                                   void* qa, void* cache, void* stream) {
+                                   int dn, int dr, int rot_dims, int interleaved, int R, int q_off, int dkv_off,
+                                   const float* norm_w, float eps, const int32_t* positions, const float* cos_sin, int max_pos,
+                                   const int64_t* slots, int bs, void* qa, void* cache, void* stream) {
     B2_REQUIRE(T >= 0 && H > 0 && dn >= 0 && dr >= 0 && R > 0 && bs > 0 && q_off >= 0 && rot_dims >= 0 && rot_dims <= dr &&
                    rot_dims % 2 == 0 && max_pos > 0, B2_EINVAL, "latent_prep: bad sizes");
     if (T == 0) return B2_OK;
@@ -966,18 +1023,19 @@ extern "C" int b2_latent_prep_rows(const void* q, int64_t q_stride, const void* 
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     const int work = H * dr > R ? H * dr : R;
     const int threads = work >= 2048 ? 256 : 128;
-    const bool vec = q_stride % 4 == 0 && q_off % 4 == 0 && dn % 4 == 0 && dr % 4 == 0 && R % 4 == 0 && rot_dims % 4 == 0 &&
+    const bool vec = q_stride % 4 == 0 && q_off % 4 == 0 && dn % 4 == 0 && dr % 4 == 0 && R % 4 == 0 &&
+                     rot_dims % (interleaved ? 4 : 8) == 0 &&
                      (dkv_off < 0 || (dkv_off % 4 == 0 && kv_stride % 4 == 0 && b2_aligned16(kv))) && b2_aligned16(q) &&
                      b2_aligned16(qa) && (dkv_off < 0 || b2_aligned16(cache));
     B2_DISPATCH_ACT(act_dtype, A, {
         if (vec)
             latent_prep_vec_kernel<A><<<T, threads, 0, st>>>(static_cast<const A*>(q), q_stride, static_cast<const A*>(kv), kv_stride,
-                                                             H, dn, dr, rot_dims, R, q_off, dkv_off, norm_w, eps, positions,
-                                                             cos_sin, max_pos, slots, static_cast<A*>(qa), static_cast<A*>(cache));
+                                                             H, dn, dr, rot_dims, interleaved != 0, R, q_off, dkv_off, norm_w,
+                                                             eps, positions, cos_sin, max_pos, slots, static_cast<A*>(qa), static_cast<A*>(cache));
         else
             latent_prep_kernel<A><<<T, threads, 0, st>>>(static_cast<const A*>(q), q_stride, static_cast<const A*>(kv), kv_stride, H,
-                                                         dn, dr, rot_dims, R, q_off, dkv_off, norm_w, eps, positions, cos_sin,
-                                                         max_pos, slots, bs, static_cast<A*>(qa), static_cast<A*>(cache));
+                                                         dn, dr, rot_dims, interleaved != 0, R, q_off, dkv_off, norm_w, eps,
+                                                         positions, cos_sin, max_pos, slots, bs, static_cast<A*>(qa), static_cast<A*>(cache));
     });
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
@@ -985,8 +1043,8 @@ extern "C" int b2_latent_prep_rows(const void* q, int64_t q_stride, const void* 
 
 extern "C" int b2_latent_attention(void* out, const void* qa, const void* cache, int act_dtype, const int32_t* block_tables,
                                    int max_nb, const int32_t* cu_q, const int32_t* ctx_start, int n_seq, int T, int H, int R,
-                                   int dr, int bs, float scale, int window, const void* gate, int64_t gate_stride,
-                                   float* workspace, int64_t workspace_floats, void* stream) {
+                                   int dr, int bs, float scale, int window, const float* sink_logits, const void* gate,
+                                   int64_t gate_stride, float* workspace, int64_t workspace_floats, void* stream) {
     B2_REQUIRE(T >= 0 && H > 0 && R > 0 && dr >= 0 && bs > 0 && window >= 0, B2_EINVAL, "latent_attention: bad sizes");
     B2_REQUIRE(R <= 32 * kMaxRPerLane, B2_EUNSUPPORTED, "latent_attention: latent size %d above %d", R, 32 * kMaxRPerLane);
     if (T == 0 || n_seq == 0) return B2_OK;
@@ -997,8 +1055,8 @@ extern "C" int b2_latent_attention(void* out, const void* qa, const void* cache,
         int nsplit = plan.nsplit;
         if (nsplit > 1 && (!workspace || workspace_floats < (int64_t)T * H * nsplit * (R + 2))) nsplit = 1;
 #define B2_LAT(RT)                                                                                                            \
-    return launch_latent_mma<RT>(out, qa, cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, dr, bs, scale, window, gate, \
-                                 gate_stride, plan.decode, nsplit, nsplit > 1 ? workspace : nullptr, st)
+    return launch_latent_mma<RT>(out, qa, cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, dr, bs, scale, window, \
+                                 sink_logits, gate, gate_stride, plan.decode, nsplit, nsplit > 1 ? workspace : nullptr, st)
         if (R == 64) B2_LAT(4);
         if (R == 128) B2_LAT(8);
         if (R == 256) B2_LAT(16);
@@ -1011,7 +1069,7 @@ extern "C" int b2_latent_attention(void* out, const void* qa, const void* cache,
     const int items = T * H, blocks = (items + warps - 1) / warps;
     B2_DISPATCH_ACT(act_dtype, A, (latent_attention_kernel<A><<<blocks, warps * 32, smem, st>>>(
         static_cast<const A*>(qa), static_cast<const A*>(cache), block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, R, dr, bs,
-        scale, window, static_cast<const A*>(gate), gate_stride, static_cast<A*>(out))));
+        scale, window, sink_logits, static_cast<const A*>(gate), gate_stride, static_cast<A*>(out))));
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }
@@ -1031,8 +1089,9 @@ extern "C" int b2_latent_gather(void* out, const void* cache, const int32_t* blo
 extern "C" int b2_window_attention(void* out, const void* qn, int64_t qn_row, int qn_head, const void* qr, int64_t qr_row,
                                    int qr_head, const void* kn, const void* kt, int64_t kt_row, const void* v,
                                    const int32_t* cu_q, const int32_t* ctx_start, const int32_t* cu_k, const int32_t* k_lo,
-                                   int n_seq, int T, int H, int dn, int dr, int dv, float scale, int window, const void* gate,
-                                   int64_t gate_stride, void* stream) {
+                                   int n_seq, int T, int H, int dn, int dr, int dv, float scale, int window,
+                                   const float* sink_logits, const void* gate, int64_t gate_stride, int gate_channels,
+                                   int64_t out_stride, void* stream) {
     B2_REQUIRE(T >= 0 && n_seq >= 0 && H > 0 && dn >= 0 && dr >= 0 && dv > 0 && window >= 0, B2_EINVAL, "window_attention: bad sizes");
     B2_REQUIRE(dn % 8 == 0 && dr % 8 == 0 && (dn + dr) % 16 == 0 && dn + dr > 0 && dv % 16 == 0 && dv <= 16 * kWMaxDVT, B2_EUNSUPPORTED,
                "window_attention: head sizes %d + %d / %d", dn, dr, dv);
@@ -1041,6 +1100,11 @@ extern "C" int b2_window_attention(void* out, const void* qn, int64_t qn_row, in
     B2_REQUIRE(b2_aligned16(out) && b2_aligned16(qn) && b2_aligned16(qr) && b2_aligned16(kn) && b2_aligned16(kt) && b2_aligned16(v) &&
                    qn_row % 8 == 0 && qn_head % 8 == 0 && qr_row % 8 == 0 && qr_head % 8 == 0 && kt_row % 8 == 0, B2_EINVAL,
                "window_attention: pointers and strides must keep 16-byte alignment");
+    B2_REQUIRE(out_stride >= (int64_t)H * dv && out_stride % 8 == 0, B2_EINVAL, "window_attention: output rows of stride %lld",
+               (long long)out_stride);
+    B2_REQUIRE(!gate || !gate_channels || (gate_stride >= (int64_t)H * dv && gate_stride % 2 == 0 &&
+                                           reinterpret_cast<uintptr_t>(gate) % 4 == 0), B2_EINVAL,
+               "window_attention: a gate per channel needs 4-byte aligned rows of H * dv columns");
     const size_t smem = (size_t)((kWQ + kWK) * (dn + dr + 8) + kWK * (dv + 8)) * sizeof(__nv_bfloat16);
     B2_REQUIRE(smem <= 200 * 1024, B2_EUNSUPPORTED, "window_attention: key size %d too large", dn + dr);
     if (smem > 48 * 1024)
@@ -1049,8 +1113,8 @@ extern "C" int b2_window_attention(void* out, const void* qn, int64_t qn_row, in
     window_attention_kernel<<<dim3(tiles, H), 128, smem, static_cast<cudaStream_t>(stream)>>>(
         static_cast<const __nv_bfloat16*>(qn), qn_row, qn_head, static_cast<const __nv_bfloat16*>(qr), qr_row, qr_head,
         static_cast<const __nv_bfloat16*>(kn), static_cast<const __nv_bfloat16*>(kt), kt_row, static_cast<const __nv_bfloat16*>(v), cu_q,
-        ctx_start, cu_k, k_lo, n_seq, H, dn, dr, dv, scale * 1.4426950408889634f, window, static_cast<const __nv_bfloat16*>(gate),
-        gate_stride, static_cast<__nv_bfloat16*>(out));
+        ctx_start, cu_k, k_lo, n_seq, H, dn, dr, dv, scale * kLog2e, window, sink_logits, static_cast<const __nv_bfloat16*>(gate),
+        gate_stride, gate_channels != 0, static_cast<__nv_bfloat16*>(out), out_stride);
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }

@@ -17,6 +17,10 @@
 //                      or gelu_tanh(g) * u, gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) (B2_GLU_GELU_TANH)
 //   b2_gate_mul        out[t, i] = x[t, i] * act(gate[t, i]) * scale with act = sigmoid (B2_GATE_SIGMOID) or SiLU
 //                      (B2_GATE_SILU): an output gate on concatenated head outputs, the three rows with strides of their own
+//   b2_parallel_join   the input row of the ONE output projection of a layer whose mixer and feed-forward run side by side on
+//                      the same norm, [ x * sigmoid(gate) | act(up) ]: gated mixer heads (for the first mix_rows rows; an
+//                      attention kernel may have written the others itself) beside the activated feed-forward units, so that
+//                      W_o and W_down are one product over the concatenated columns and their sum never leaves its accumulator.
 //   b2_softcap         z <- cap * tanh(z / cap) in place
 // The residual and all statistics are fp32 whatever the activation type.
 #include "b2_act.cuh"
@@ -220,6 +224,35 @@ __global__ void gate_mul_kernel(T* __restrict__ out, int64_t out_stride, const T
     }
 }
 
+template <typename T, int W>
+__global__ void __launch_bounds__(256)
+parallel_join_kernel(T* __restrict__ out, int64_t out_stride, const T* __restrict__ x, int64_t x_stride, const T* __restrict__ gate,
+                     int64_t gate_stride, int mix_rows, int n_mix, const T* __restrict__ up, int64_t up_stride, int n_ff, int act,
+                     float a, float b) {
+    const int t = blockIdx.x;
+    const int first = t < mix_rows ? 0 : n_mix;
+    T* o = out + (size_t)t * out_stride;
+    for (int i = first + (blockIdx.y * blockDim.x + threadIdx.x) * W; i < n_mix + n_ff; i += gridDim.y * blockDim.x * W) {
+        float v[4] = {0.f, 0.f, 0.f, 0.f}, z[4] = {0.f, 0.f, 0.f, 0.f};
+        if (i < n_mix) {
+            const T* xs = x + (size_t)t * x_stride + i;
+            if (W == 4) b2::ld4(xs, v); else v[0] = b2::ld(xs);
+            if (gate) {
+                const T* gs = gate + (size_t)t * gate_stride + i;
+                if (W == 4) b2::ld4(gs, z); else z[0] = b2::ld(gs);
+#pragma unroll
+                for (int c = 0; c < W; ++c) v[c] *= b2::sigmoid_f(z[c]);
+            }
+        } else {
+            const T* us = up + (size_t)t * up_stride + (i - n_mix);
+            if (W == 4) b2::ld4(us, z); else z[0] = b2::ld(us);
+#pragma unroll
+            for (int c = 0; c < W; ++c) v[c] = act == B2_FF_XIELU ? b2::xielu_f(z[c], a, b) : b2::relu_sq_f(z[c]);
+        }
+        if (W == 4) b2::st4(o + i, v); else b2::st(o + i, v[0]);
+    }
+}
+
 template <typename T>
 __global__ void softcap_kernel(T* __restrict__ z, int64_t stride, int V, float cap) {
     const int t = blockIdx.x;
@@ -341,6 +374,36 @@ extern "C" int b2_gate_mul(void* out, int64_t out_stride, const void* x, int64_t
                                                                            kind, scale);
         else gate_mul_kernel<A, 1><<<rows_grid(I, T), 256, 0, st>>>(static_cast<A*>(out), out_stride, static_cast<const A*>(x),
                                                                    x_stride, static_cast<const A*>(gate), gate_stride, I, kind, scale);
+    });
+    B2_CUDA_OK(cudaGetLastError());
+    return B2_OK;
+}
+
+extern "C" int b2_parallel_join(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* gate,
+                                int64_t gate_stride, int mix_rows, int n_mix, const void* up, int64_t up_stride, int n_ff,
+                                int ff_act, float act_a, float act_b, int act_dtype, int T, void* stream) {
+    B2_REQUIRE(T >= 0 && mix_rows >= 0 && mix_rows <= T && n_mix >= 0 && n_ff >= 0 && n_mix + n_ff > 0 && out_stride >= n_mix + n_ff,
+               B2_EINVAL, "parallel_join: bad sizes T=%d mix=%d ff=%d", T, n_mix, n_ff);
+    B2_REQUIRE(ff_act == B2_FF_XIELU || ff_act == B2_FF_RELU_SQ, B2_EINVAL, "parallel_join: unknown activation %d", ff_act);
+    if (T == 0 || (n_ff == 0 && mix_rows == 0)) return B2_OK;
+    B2_REQUIRE(out && (n_ff == 0 || up) && (mix_rows == 0 || n_mix == 0 || x), B2_EINVAL, "parallel_join: null pointer");
+    if (n_ff == 0) T = mix_rows;                                  // nothing to do for the other rows
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const size_t esz = act_dtype == B2_ACT_BF16 ? 2 : 4;
+    auto ok = [&](const void* p, int64_t stride) { return !p || (stride % 4 == 0 && reinterpret_cast<uintptr_t>(p) % (4 * esz) == 0); };
+    const bool vec = n_mix % 4 == 0 && n_ff % 4 == 0 && ok(out, out_stride) && ok(x, x_stride) && ok(gate, gate_stride) &&
+                     ok(up, up_stride);
+    const int cols = n_mix + n_ff;
+    B2_DISPATCH_ACT(act_dtype, A, {
+        A* o = static_cast<A*>(out);
+        const A* xs = static_cast<const A*>(x);
+        const A* gs = static_cast<const A*>(gate);
+        const A* us = static_cast<const A*>(up);
+        if (vec) parallel_join_kernel<A, 4><<<rows_grid(cols / 4, T), 256, 0, st>>>(o, out_stride, xs, x_stride, gs, gate_stride,
+                                                                                    mix_rows, n_mix, us, up_stride, n_ff, ff_act,
+                                                                                    act_a, act_b);
+        else parallel_join_kernel<A, 1><<<rows_grid(cols, T), 256, 0, st>>>(o, out_stride, xs, x_stride, gs, gate_stride, mix_rows,
+                                                                            n_mix, us, up_stride, n_ff, ff_act, act_a, act_b);
     });
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
