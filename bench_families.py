@@ -1,9 +1,10 @@
-"""`bench.py --family kofadra|gatolix|tonilix|sanarax`: prefill and decode throughput of a model family at layer sizes of real models
+"""`bench.py --family kofadra|gatolix|tonilix|sanarax|gapidra`: prefill and decode throughput of a model family at layer sizes of real models
 (random weights), beside the Llama model of equal width, heads, head size and ACTIVE feed-forward width, plus the device
 time of every kernel of the family with the roofline that bounds it beside the like kernel of the Llama path (Tonilix:
 beside the Kofadra family, whose recurrent mixer, attention without rotation and routed experts are the closest; Sanarax:
 beside the Gatolix family, whose norms on both sides, latent attention and squared-ReLU feed-forward are the closest, with
-the like kernel of Kofadra and Tonilix for the sink attention and the linear attention).
+the like kernel of Kofadra and Tonilix for the sink attention and the linear attention; Gapidra: beside Sanarax, whose
+windowed grouped-query attention, latent attention and dense ungated feed-forward are the closest).
 
 Both models run through the same engine (LLMEngine.replay_step: scheduler, pools, state slots, CUDA-graph decode).
   prefill   one prompt chunk of T tokens in one step; wall clock around the step (it ends with a stream synchronize)
@@ -43,6 +44,10 @@ SANARAX_SIZES = {
     "4k": dict(hidden=4096, layers=6, heads=32, kv_heads=8, head_dim=128, ff=14336, vocab=32000, kv_rank=512, q_rank=1536,
                rot_dim=64, window=1024, keep_first=4),
 }
+
+
+# Gapidra: the same widths, heads and latent; latent and sigmoid-attention layers in turn (no query latent)
+GAPIDRA_SIZES = {k: dict({n: v for n, v in s.items() if n not in ("q_rank", "keep_first")}, layers=6) for k, s in SANARAX_SIZES.items()}
 
 
 def _peaks():
@@ -619,10 +624,130 @@ def _kernels_sanarax(size, s, B, ctx, T):
         torch.cuda.empty_cache()
 
 
+def _kernels_gapidra(size, s, B, ctx, T):
+    """Device time of the kernels of a Gapidra layer, each beside the like kernel of Sanarax (or Gatolix, Llama) on the same
+    shapes."""
+    import torch
+    from b200attn import ops
+    dev = torch.device("cuda", 0)
+    HBM, TF, src = _peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    D, H, G, d, F, W, R, dr = (s[k] for k in ("hidden", "heads", "kv_heads", "head_dim", "ff", "window", "kv_rank", "rot_dim"))
+    Dc, bf = R + dr, torch.bfloat16
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)          # noqa: E731
+
+    def line(kernel, phase, ms, bytes_=0, flops=0, like=None):
+        gbs, tfs = bytes_ / ms / 1e6, flops / ms / 1e9
+        _emit(bench="kernel", size=size, kernel=kernel, phase=phase, ms=round(ms, 4), gb_per_s=round(gbs, 1),
+              tflop_per_s=round(tfs, 2), frac_hbm=round(gbs / HBM, 3), frac_bf16=round(tfs / TF, 4), peaks=src, like=like)
+
+    yarn = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    tab_s = ops.rotary_table(ctx + T + 64, d // 2, 1e6, yarn, dev)
+    tab_l = ops.rotary_table(ctx + T + 64, dr, 1e4, None, dev)
+    for phase, n_seq, q_len, c in (("prefill", 1, T, 0), ("decode", B, 1, ctx)):
+        rows = n_seq * q_len
+        nb_seq = (c + q_len + 15) // 16
+        tables = torch.arange(n_seq * nb_seq, dtype=torch.int32, device=dev).view(n_seq, nb_seq)
+        batch = ops.SeqBatch(i32([i * q_len for i in range(n_seq + 1)]), i32([c] * n_seq), tables, None, n_seq, rows)
+        pos = (torch.arange(rows, device=dev) % q_len + c).to(torch.int32)
+        slots = (torch.arange(rows, device=dev) // q_len * (nb_seq * 16) + pos).to(torch.int64)
+        pairs = sum(min(p + 1, W) for p in range(T))
+        seen = min(c + 1, W)
+        # ---- residual add + the next layer's RMS norm  |  like: Sanarax's norms on both sides
+        x, y = torch.randn(rows, D, device=dev), torch.randn(rows, D, device=dev).to(bf)
+        one = torch.ones(D, device=dev)
+        ms = _time(lambda: ops.sandwich_norm(x, y, pre_w=one, eps=1e-6, norm_kind=ops.NORM_RMS), flush)
+        line("sandwich_norm (residual add + RMS norm)", phase, ms, bytes_=rows * D * 12, like="sandwich_norm (Sanarax)")
+        ms = _time(lambda: ops.sandwich_norm(x, y, one, None, one, None, eps=1e-6, norm_kind=ops.NORM_RMS), flush)
+        line("sandwich_norm (Sanarax, 2 RMS norms)", phase, ms, bytes_=rows * D * 12)
+        # ---- the two products of a layer (library GEMMs): all that reads the norm, all that is added to the residual
+        for kind, n_in, n_mix in (("latent", H * (2 * d + dr) + Dc, H * d), ("attention", (H + 2 * G) * d, H * d)):
+            h = torch.randn(rows, D, device=dev).to(bf)
+            w_in = torch.randn(n_in + F, D, device=dev).to(bf)
+            w_out = torch.randn(D, n_mix + F, device=dev).to(bf)
+            j = torch.randn(rows, n_mix + F, device=dev).to(bf)
+            lin = torch.nn.functional.linear
+            ms = _time(lambda: (lin(h, w_in), lin(j, w_out)), flush)
+            par = D * (n_in + n_mix + 2 * F)
+            io = 2 * (par + rows * (2 * D + n_in + n_mix + 2 * F))
+            line(f"products of a {kind} layer (2 cuBLAS GEMMs, mixer and feed-forward together)", phase, ms, flops=2 * rows * par,
+                 bytes_=io, like=f"products of a {kind} layer (4 GEMMs)")
+            wa, wb, wc, wd = w_in[:n_in], w_in[n_in:], w_out[:, :n_mix].contiguous(), w_out[:, n_mix:].contiguous()
+            ja, jb = j[:, :n_mix].contiguous(), j[:, n_mix:].contiguous()
+            ms = _time(lambda: (lin(h, wa), lin(ja, wc), lin(h, wb), lin(jb, wd)), flush)
+            line(f"products of a {kind} layer (4 GEMMs, mixer and feed-forward apart)", phase, ms, flops=2 * rows * par, bytes_=io)
+            del w_in, w_out, h, j, ja, jb, wa, wb, wc, wd
+        # ---- joint input of the output projection  |  like: Sanarax's squared ReLU (and, for the gate, gate_mul)
+        Pl = H * (2 * d + dr) + Dc + F
+        proj = torch.randn(rows, Pl, device=dev).to(bf)
+        up, gate = proj[:, Pl - F:], proj[:, H * (d + dr):H * (2 * d + dr)]
+        joint = torch.empty(rows, H * d + F, dtype=bf, device=dev)
+        ms = _time(lambda: ops.parallel_join(joint, None, None, H * d, up, ops.FF_XIELU, 0.7, 1.2), flush)
+        line("parallel_join (xIELU columns)", phase, ms, bytes_=rows * F * 4, like="relu_sq (Sanarax)")
+        act = torch.randn(rows, F, device=dev).to(bf)
+        ms = _time(lambda: ops.relu_sq(act), flush)
+        line("relu_sq (Sanarax)", phase, ms, bytes_=rows * F * 4)
+        heads = torch.randn(rows, H * d, device=dev).to(bf)
+        ms = _time(lambda: ops.parallel_join(joint, heads, gate, H * d, up, ops.FF_XIELU, 0.7, 1.2), flush)
+        line("parallel_join (gated heads + xIELU columns)", phase, ms, bytes_=rows * (F * 4 + H * d * 6), like="gate_mul + relu_sq")
+        gm = torch.randn(rows, H * d, device=dev).to(bf)
+        ms = _time(lambda: (ops.gate_mul(heads, gm), ops.relu_sq(act)), flush)
+        line("gate_mul + relu_sq (Tonilix, Sanarax)", phase, ms, bytes_=rows * (F * 4 + H * d * 6))
+        # ---- sigmoid attention: whole-projection norms + rotation + pool write  |  like: Sanarax's rotation + pool write
+        kc = torch.randn(n_seq * nb_seq, G, 16, d, device=dev).to(bf)
+        vc = torch.randn(n_seq * nb_seq, G, 16, d, device=dev).to(bf)
+        qkv = torch.randn(rows, (H + 2 * G) * d + F, device=dev).to(bf)
+        nq, nk = torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+        io = rows * (2 * H + 4 * G) * d * 2
+        ms = _time(lambda: ops.qk_rope_cache(qkv, H, G, d, d, pos, tab_s, d // 2, slots, kc, vc, interleaved=True, q_norm=nq, k_norm=nk), flush)
+        line("qk_norm_rope_cache (whole-projection norms, half of every head turns)", phase, ms, bytes_=io, like="qk_rope_cache (Sanarax)")
+        ms = _time(lambda: ops.qk_rope_cache(qkv, H, G, d, d, pos, tab_s, d // 2, slots, kc, vc, v_from_k=True), flush)
+        line("qk_rope_cache (Sanarax)", phase, ms, bytes_=rows * (2 * H + 3 * G) * d * 2)
+        q = torch.randn(rows, H, d, device=dev).to(bf)
+        pb, sinks = torch.full((H,), -4.0, device=dev), torch.randn(H, device=dev)
+        hg = torch.randn(rows, H, device=dev).to(bf)
+        ms = _time(lambda: ops.chunk_attention(q, kc, vc, batch, d ** -0.5, window=W, weight_kind=ops.WEIGHT_SIGMOID, head_bias=pb,
+                                               out=joint[:, :H * d]), flush)
+        work = dict(flops=4 * pairs * H * d) if phase == "prefill" else dict(bytes_=n_seq * seen * G * 2 * d * 2)
+        line("chunk_attention (sigmoid weights, window %d)" % W, phase, ms, like="chunk_attention (Sanarax)", **work)
+        ms = _time(lambda: ops.chunk_attention(q, kc, vc, batch, d ** -0.5, window=W, sink=1.0, sink_logits=sinks, gate=hg), flush)
+        line("chunk_attention (Sanarax: softmax, sink, gate, window %d)" % W, phase, ms, **work)
+        # ---- latent attention: prep, then the attention of the phase  |  like: Gatolix's and Sanarax's (no sink, gate per head)
+        cache = torch.randn(n_seq * nb_seq, 16, Dc, device=dev).to(bf)
+        nw = torch.ones(R, device=dev)
+        dkv = H * (2 * d + dr)
+        io = rows * (H * dr * 4 + Dc * 4)
+        ms = _time(lambda: ops.latent_prep(proj, H, d, dr, dr, R, 0, dkv, nw, 1e-6, pos, tab_l, slots, cache, interleaved=False), flush)
+        line("latent_prep (half layout)", phase, ms, bytes_=io, like="latent_prep (Gatolix)")
+        ms = _time(lambda: ops.latent_prep(proj, H, d, dr, dr, R, 0, dkv, nw, 1e-6, pos, tab_l, slots, cache), flush)
+        line("latent_prep (Gatolix, interleaved)", phase, ms, bytes_=io)
+        qa = torch.randn(rows, H, Dc, device=dev).to(bf)
+        if phase == "prefill":
+            cu, cs = i32([0, T]), i32([0])
+            lat = ops.latent_gather(cache, tables, cu, cs, 1, T)
+            kn, vb = torch.randn(T, H, d, device=dev).to(bf), torch.randn(T, H, d, device=dev).to(bf)
+            q3 = proj[:, :H * (d + dr)].view(rows, H, d + dr)
+            args = (q3[:, :, :d], qa[:, :, R:], kn, lat[:, R:], vb, cu, cs, cu, cs, 1, 0.07, W)
+            ms = _time(lambda: ops.window_attention(*args, gate=gate, sink_logits=sinks, out=joint[:, :H * d]), flush)
+            line("window_attention (per-head keys, window %d, sink, gate per channel)" % W, phase, ms, flops=2 * pairs * H * (2 * d + dr),
+                 like="window_attention (Gatolix)")
+            ms = _time(lambda: ops.window_attention(*args, gate=hg), flush)
+            line("window_attention (Gatolix, window %d, gate per head)" % W, phase, ms, flops=2 * pairs * H * (2 * d + dr))
+        else:
+            io = n_seq * seen * Dc * 2 + rows * H * (Dc + R) * 2
+            ms = _time(lambda: ops.latent_attention(qa, cache, batch, R, 0.07, W, sink_logits=sinks), flush)
+            line("latent_attention (window %d, sink)" % W, phase, ms, bytes_=io, flops=2 * n_seq * seen * H * (Dc + R),
+                 like="latent_attention (Gatolix)")
+            ms = _time(lambda: ops.latent_attention(qa, cache, batch, R, 0.07, W, gate=hg), flush)
+            line("latent_attention (Gatolix, window %d)" % W, phase, ms, bytes_=io, flops=2 * n_seq * seen * H * (Dc + R))
+        del kc, vc, cache, proj, joint, qkv, qa
+        torch.cuda.empty_cache()
+
+
 def run(family: str, sizes, steps: int, kernels: bool = True) -> None:
     import torch
     from b200attn.model import ModelConfig
-    if family not in ("kofadra", "gatolix", "tonilix", "sanarax"):
+    if family not in ("kofadra", "gatolix", "tonilix", "sanarax", "gapidra"):
         raise SystemExit(f"unknown family {family!r}")
     B, ctx, T = 64, 2560, 4096          # ctx: 2.5 mask blocks / windows of the bench geometries
     for name in sizes:
@@ -642,6 +767,11 @@ def run(family: str, sizes, steps: int, kernels: bool = True) -> None:
             fcfg = bench_config(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["head_dim"], s["ff"], s["vocab"],
                                 kv_rank=s["kv_rank"], q_rank=s["q_rank"], rot_dim=s["rot_dim"], window=s["window"],
                                 keep_first=s["keep_first"], name=f"sanarax-{name}")
+        elif family == "gapidra":
+            from b200attn.gapidra import bench_config
+            s = GAPIDRA_SIZES[name]
+            fcfg = bench_config(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["head_dim"], s["ff"], s["vocab"],
+                                kv_rank=s["kv_rank"], rot_dim=s["rot_dim"], window=s["window"], name=f"gapidra-{name}")
         else:
             from b200attn.gatolix import bench_config
             s = GATOLIX_SIZES[name]
@@ -663,8 +793,15 @@ def run(family: str, sizes, steps: int, kernels: bool = True) -> None:
             gcfg = gatolix_config(s["hidden"], s["layers"], s["heads"], s["head_dim"], s["rot_dim"], s["head_dim"], s["kv_rank"],
                                   g["ff"], g["experts"], g["top"], s["vocab"], window=s["window"], name=f"gatolix-{name}")
             _throughput(gcfg.name, gcfg, B, ctx, T, steps)
+        if family == "gapidra":                 # the closest family at equal size: windowed and latent attention, dense feed-forwards
+            from b200attn.sanarax import bench_config as sanarax_config
+            g = SANARAX_SIZES[name]
+            scfg = sanarax_config(g["hidden"], g["layers"], g["heads"], g["kv_heads"], g["head_dim"], g["ff"], g["vocab"],
+                                  kv_rank=g["kv_rank"], q_rank=g["q_rank"], rot_dim=g["rot_dim"], window=g["window"],
+                                  keep_first=g["keep_first"], name=f"sanarax-{name}")
+            _throughput(scfg.name, scfg, B, ctx, T, steps)
         _throughput(lcfg.name, lcfg, B, ctx, T, steps)
         if kernels:
             {"kofadra": _kernels_kofadra, "gatolix": _kernels_gatolix, "tonilix": _kernels_tonilix,
-             "sanarax": _kernels_sanarax}[family](name, s, B, ctx, T)
+             "sanarax": _kernels_sanarax, "gapidra": _kernels_gapidra}[family](name, s, B, ctx, T)
         torch.cuda.empty_cache()

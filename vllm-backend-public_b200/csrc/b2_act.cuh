@@ -53,9 +53,24 @@ __device__ __forceinline__ float relu_sq_f(float z) {
     z = fmaxf(z, 0.f);
     return z * z;
 }
+// The functions of an epilogue at the precision of the type it stores: float takes the accurate forms, bf16 (8 bits of
+// mantissa) the hardware exponential and reciprocal, whose error is far below what it keeps.
+template <typename T>
+__device__ __forceinline__ float sigmoid_as(float z) { return sigmoid_f(z); }
+template <>
+__device__ __forceinline__ float sigmoid_as<__nv_bfloat16>(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+// e^z - 1 - z for z <= 0; near zero, where the difference cancels, the first terms of its series
+template <typename T>
+__device__ __forceinline__ float exp_tail_as(float z) { return expm1f(z) - z; }
+template <>
+__device__ __forceinline__ float exp_tail_as<__nv_bfloat16>(float z) {
+    const float series = z * z * fmaf(z, fmaf(z, 1.f / 24.f, 1.f / 6.f), 0.5f);
+    return z > -0.125f ? series : __expf(z) - 1.f - z;
+}
 // quadratic above zero, exponential below, plus half the identity: a z^2 + z/2, b (e^z - 1 - z) + z/2
-__device__ __forceinline__ float xielu_f(float z, float a, float b) {
-    return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (expm1f(z) - z));
+template <typename T>
+__device__ __forceinline__ float xielu_as(float z, float a, float b) {
+    return fmaf(0.5f, z, z > 0.f ? a * z * z : b * exp_tail_as<T>(z));
 }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
@@ -74,6 +89,20 @@ __device__ __forceinline__ void st4(float* p, const float (&v)[4]) {
 }
 __device__ __forceinline__ void st4(__nv_bfloat16* p, const float (&v)[4]) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+
+// eight consecutive elements of a bf16 row (16 bytes, aligned)
+__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 t = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {t.x, t.y, t.z, t.w};
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+        v[2 * c] = __uint_as_float(w[c] << 16);
+        v[2 * c + 1] = __uint_as_float(w[c] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void st8(__nv_bfloat16* p, const float (&v)[8]) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
 }
 
 // Sequence of batch row `row` when rows are grouped by cu[0..n] (cu[0] = 0, cu[n] = rows in the batch).

@@ -68,8 +68,21 @@ __device__ __forceinline__ void qk_row_scales(const T* src, int nq, int nk, floa
         for (int c = 0; c < W; ++c) ss = fmaf(v[c], v[c], ss);
         if (i < nq) sq += ss; else sk += ss;
     }
-    inv_q = rsqrtf(b2::block_sum(sq, red) / (float)nq + eps);
-    inv_k = rsqrtf(b2::block_sum(sk, red) / (float)nk + eps);
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    sq = b2::warp_sum(sq);
+    sk = b2::warp_sum(sk);
+    if (lane == 0) {
+        red[2 * wid] = sq;
+        red[2 * wid + 1] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int x = 0; x < nw; ++x) {                   // at most eight warps: every thread adds them up itself
+        sq += red[2 * x];
+        sk += red[2 * x + 1];
+    }
+    inv_q = rsqrtf(sq / (float)nq + eps);
+    inv_k = rsqrtf(sk / (float)nk + eps);
 }
 
 // Rows [q | k] (+ [v]): partial rotation of the q and k heads, K (rotated) and V pool writes; see the file comment.  NORM:
@@ -80,7 +93,7 @@ __global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stri
                                      const float* __restrict__ cos_sin, int max_pos, const int64_t* __restrict__ slots, int bs,
                                      const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                                      T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache) {
-    __shared__ float red[33];
+    __shared__ float red[16];
     const int row = blockIdx.x;
     const T* src = qkv + (size_t)row * qkv_stride;
     float inv_q = 1.f, inv_k = 1.f;
@@ -128,7 +141,7 @@ qk_rope_cache_vec_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, i
                          bool interleaved, const int32_t* __restrict__ positions, const float* __restrict__ cos_sin, int max_pos,
                          const int64_t* __restrict__ slots, int bs, const float* __restrict__ q_w, const float* __restrict__ k_w,
                          float eps, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache) {
-    __shared__ float red[33];
+    __shared__ float red[16];
     const int row = blockIdx.x;
     const T* src = qkv + (size_t)row * qkv_stride;
     float inv_q = 1.f, inv_k = 1.f;
@@ -236,7 +249,7 @@ __global__ void qknorm_cache_kernel(const T* __restrict__ qkv, int64_t qkv_strid
 }
 
 // sigmoid of a score that is already in the exponent of 2
-__device__ __forceinline__ float sigmoid2_f(float x2) { return __fdividef(1.f, 1.f + exp2f(-x2)); }
+__device__ __forceinline__ float sigmoid2_f(float x2) { return __fdividef(1.f, 1.f + b2::fast_exp2(-x2)); }
 
 template <typename T, bool SIG>
 __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
@@ -511,10 +524,12 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
 // ------------------------------------------------------------------------------------------------- tiled prompt kernel
 // bf16, dk and dv multiples of 16: one CTA = 64 consecutive query rows of one sequence x one head, four warps of 16 rows.
 // Keys are walked 64 at a time from the first row's block start to the last row's position (at most chunk + 63 keys
-// with a mask, the whole prefix without): K and V tiles are gathered from the pages into shared memory, S = Q K^T and
+// with a mask, the whole prefix without): K and V tiles are gathered from the pages into shared memory (cp.async, two
+// threads per key row with one page lookup each, the next tile in flight while this one is multiplied), S = Q K^T and
 // O += P V run on mma.sync m16n8k16 with ldmatrix operands, the online softmax lives in the accumulator registers
-// (exp2 with the scale folded in, the sink seeding the running maximum and denominator).  Sequences with fewer than
-// kTileMinRows rows (decode rows) are left to the warp kernel above.
+// (exp2 with the scale folded in, the sink seeding the running maximum and denominator).  A warp tests the mask per score
+// only in tiles that its rows see in part.  Sequences with fewer than kTileMinRows rows (decode rows) are left to the warp
+// kernel above.
 constexpr int kTQ = 64, kTK = 64, kTileMinRows = 16;
 
 template <int DKT, int DVT, bool SIG>
@@ -529,8 +544,8 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     constexpr int DK = 16 * DKT, DV = 16 * DVT, LDK = DK + 8, LDV = DV + 8;
     extern __shared__ __align__(16) unsigned char tile_smem[];
     __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(tile_smem);      // [64][LDK]
-    __nv_bfloat16* k_sm = q_sm + kTQ * LDK;                                 // [64][LDK]
-    __nv_bfloat16* v_sm = k_sm + kTK * LDK;                                 // [64][LDV]
+    __nv_bfloat16* k_sm = q_sm + kTQ * LDK;                                 // [2][64][LDK]
+    __nv_bfloat16* v_sm = k_sm + 2 * kTK * LDK;                             // [2][64][LDV]
     __shared__ int s_info[2];
     const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
     if (tid == 0) {
@@ -575,109 +590,148 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     float o[2 * DVT][4];
 #pragma unroll
     for (int n = 0; n < 2 * DVT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
-    const uint32_t q_base = b2::smem_u32(q_sm), k_base = b2::smem_u32(k_sm), v_base = b2::smem_u32(v_sm);
+    const uint32_t q_base = b2::smem_u32(q_sm), k_base0 = b2::smem_u32(k_sm), v_base0 = b2::smem_u32(v_sm);
 
-    for (int kv0 = 0; kv0 < span.n; kv0 += kTK) {                           // kv0: compact key index of the tile's first key
-        __syncthreads();                                                    // the previous tile is consumed (and Q is stored)
-        for (int idx = tid; idx < kTK * (DK / 8); idx += 128) {
-            const int key = idx / (DK / 8), c = (idx % (DK / 8)) * 8, j = span.key(kv0 + key);
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (j <= p_last) v = *reinterpret_cast<const uint4*>(k_cache + (((size_t)bt[j / bs] * G + g) * bs + j % bs) * DK + c);
-            *reinterpret_cast<uint4*>(k_sm + key * LDK + c) = v;
-        }
-        for (int idx = tid; idx < kTK * (DV / 8); idx += 128) {
-            const int key = idx / (DV / 8), c = (idx % (DV / 8)) * 8, j = span.key(kv0 + key);
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (j <= p_last) v = *reinterpret_cast<const uint4*>(v_cache + (((size_t)bt[j / bs] * G + g) * bs + j % bs) * DV + c);
-            *reinterpret_cast<uint4*>(v_sm + key * LDV + c) = v;
-        }
-        __syncthreads();
-        {   // nothing in this tile is visible to the warp's rows: all keys after them, or all before their windows and not kept
-            const int j_min = span.key(kv0), j_max = span.key(min(kv0 + kTK, span.n) - 1);
-            if (j_min > w_last || (j_max < w_lo && (window <= 0 || j_min >= keep_first))) continue;
-        }
-        float sc[8][4];
+    const int ld_key = tid >> 1, ld_half = tid & 1;
+    auto issue = [&](int kv0, int buf) {                                    // kv0: compact key index of the tile's first key
+        const int j = span.key(kv0 + ld_key);
+        __nv_bfloat16* kd = k_sm + (buf * kTK + ld_key) * LDK;
+        __nv_bfloat16* vd = v_sm + (buf * kTK + ld_key) * LDV;
+        if (j <= p_last) {
+            const int page = j / bs;
+            const size_t row = ((size_t)bt[page] * G + g) * bs + (j - page * bs);
+            const __nv_bfloat16* ks = k_cache + row * DK;
+            const __nv_bfloat16* vs = v_cache + row * DV;
 #pragma unroll
-        for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+            for (int c = 0; c < DKT; ++c) cp_async16(kd + (2 * c + ld_half) * 8, ks + (2 * c + ld_half) * 8);
 #pragma unroll
-        for (int kk = 0; kk < DKT; ++kk) {
-            uint32_t a0, a1, a2, a3;
-            b2::ldmatrix_x4(q_base + 2u * ((w * 16 + (lane & 15)) * LDK + kk * 16 + (lane >> 4) * 8), a0, a1, a2, a3);
-#pragma unroll
-            for (int n2 = 0; n2 < 4; ++n2) {
-                uint32_t b0, b1, b2_, b3;
-                const int key = n2 * 16 + (lane >> 4) * 8 + (lane & 7), dim = kk * 16 + ((lane >> 3) & 1) * 8;
-                b2::ldmatrix_x4(k_base + 2u * (key * LDK + dim), b0, b1, b2_, b3);
-                b2::mma_bf16_16816(sc[2 * n2], a0, a1, a2, a3, b0, b1);
-                b2::mma_bf16_16816(sc[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
-            }
-        }
-        if (SIG) {                                                          // every weight by itself: nothing to rescale
-#pragma unroll
-            for (int n = 0; n < 8; ++n) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
-                    const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
-                    sc[n][e] = ok ? sigmoid2_f(fmaf(sc[n][e], scale_log2, bias_log2)) : 0.f;
-                }
-            }
+            for (int c = 0; c < DVT; ++c) cp_async16(vd + (2 * c + ld_half) * 8, vs + (2 * c + ld_half) * 8);
         } else {
-            float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
-            for (int n = 0; n < 8; ++n) {
+            for (int c = 0; c < DKT; ++c) *reinterpret_cast<uint4*>(kd + (2 * c + ld_half) * 8) = make_uint4(0, 0, 0, 0);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
-                    const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
-                    sc[n][e] = ok ? sc[n][e] * scale_log2 : -INFINITY;
+            for (int c = 0; c < DVT; ++c) *reinterpret_cast<uint4*>(vd + (2 * c + ld_half) * 8) = make_uint4(0, 0, 0, 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    issue(0, 0);
+    for (int kv0 = 0, buf = 0; kv0 < span.n; kv0 += kTK, buf ^= 1) {
+        if (kv0 + kTK < span.n) {
+            issue(kv0 + kTK, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();                                                    // the tile (and, first time, Q) is in shared memory
+        const uint32_t k_base = k_base0 + (uint32_t)(buf * kTK * LDK) * 2u, v_base = v_base0 + (uint32_t)(buf * kTK * LDV) * 2u;
+        const int j_min = span.key(kv0), j_max = span.key(min(kv0 + kTK, span.n) - 1);
+        // nothing in this tile is visible to the warp's rows: all keys after them, or all before their windows and not kept
+        const bool none = j_min > w_last || (j_max < w_lo && (window <= 0 || j_min >= keep_first));
+        // all of it is visible to all of them
+        const bool full = kv0 + kTK <= span.n && j_max <= w_first && (chunk <= 0 || j_min >= (w_last / chunk) * chunk) &&
+                          (window <= 0 || w_last - j_min < window || j_max < keep_first);
+        if (!none) {
+            float sc[8][4];
+#pragma unroll
+            for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+#pragma unroll
+            for (int kk = 0; kk < DKT; ++kk) {
+                uint32_t a0, a1, a2, a3;
+                b2::ldmatrix_x4(q_base + 2u * ((w * 16 + (lane & 15)) * LDK + kk * 16 + (lane >> 4) * 8), a0, a1, a2, a3);
+#pragma unroll
+                for (int n2 = 0; n2 < 4; ++n2) {
+                    uint32_t b0, b1, b2_, b3;
+                    const int key = n2 * 16 + (lane >> 4) * 8 + (lane & 7), dim = kk * 16 + ((lane >> 3) & 1) * 8;
+                    b2::ldmatrix_x4(k_base + 2u * (key * LDK + dim), b0, b1, b2_, b3);
+                    b2::mma_bf16_16816(sc[2 * n2], a0, a1, a2, a3, b0, b1);
+                    b2::mma_bf16_16816(sc[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
                 }
-                mx0 = fmaxf(mx0, fmaxf(sc[n][0], sc[n][1]));
-                mx1 = fmaxf(mx1, fmaxf(sc[n][2], sc[n][3]));
             }
-            mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-            mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-            mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-            mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-            const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-            const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
-            const float c0 = exp2f(m0 - mu0), c1 = exp2f(m1 - mu1);             // exp2(-inf) = 0: nothing accumulated yet
-            m0 = mn0;
-            m1 = mn1;
-            float s0 = 0.f, s1 = 0.f;
+            if (SIG) {                                                          // every weight by itself: nothing to rescale
 #pragma unroll
-            for (int n = 0; n < 8; ++n) {
-                sc[n][0] = exp2f(sc[n][0] - mu0);
-                sc[n][1] = exp2f(sc[n][1] - mu0);
-                sc[n][2] = exp2f(sc[n][2] - mu1);
-                sc[n][3] = exp2f(sc[n][3] - mu1);
-                s0 += sc[n][0] + sc[n][1];
-                s1 += sc[n][2] + sc[n][3];
+                for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) sc[n][e] = sigmoid2_f(fmaf(sc[n][e], scale_log2, bias_log2));
+                }
+                if (!full) {
+#pragma unroll
+                    for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
+                            const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
+                            if (!ok) sc[n][e] = 0.f;
+                        }
+                    }
+                }
+            } else {
+                float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+                for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) sc[n][e] *= scale_log2;
+                }
+                if (!full) {
+#pragma unroll
+                    for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
+                            const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
+                            if (!ok) sc[n][e] = -INFINITY;
+                        }
+                    }
+                }
+#pragma unroll
+                for (int n = 0; n < 8; ++n) {
+                    mx0 = fmaxf(mx0, fmaxf(sc[n][0], sc[n][1]));
+                    mx1 = fmaxf(mx1, fmaxf(sc[n][2], sc[n][3]));
+                }
+                mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+                mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+                mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+                mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+                const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
+                const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
+                const float c0 = b2::fast_exp2(m0 - mu0), c1 = b2::fast_exp2(m1 - mu1);             // exp2(-inf) = 0: nothing accumulated yet
+                m0 = mn0;
+                m1 = mn1;
+                float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+                for (int n = 0; n < 8; ++n) {
+                    sc[n][0] = b2::fast_exp2(sc[n][0] - mu0);
+                    sc[n][1] = b2::fast_exp2(sc[n][1] - mu0);
+                    sc[n][2] = b2::fast_exp2(sc[n][2] - mu1);
+                    sc[n][3] = b2::fast_exp2(sc[n][3] - mu1);
+                    s0 += sc[n][0] + sc[n][1];
+                    s1 += sc[n][2] + sc[n][3];
+                }
+                l0 = l0 * c0 + s0;
+                l1 = l1 * c1 + s1;
+#pragma unroll
+                for (int n = 0; n < 2 * DVT; ++n) {
+                    o[n][0] *= c0;
+                    o[n][1] *= c0;
+                    o[n][2] *= c1;
+                    o[n][3] *= c1;
+                }
             }
-            l0 = l0 * c0 + s0;
-            l1 = l1 * c1 + s1;
 #pragma unroll
-            for (int n = 0; n < 2 * DVT; ++n) {
-                o[n][0] *= c0;
-                o[n][1] *= c0;
-                o[n][2] *= c1;
-                o[n][3] *= c1;
+            for (int ks = 0; ks < 4; ++ks) {
+                const uint32_t a0 = b2::pack_bf16x2(sc[2 * ks][0], sc[2 * ks][1]), a1 = b2::pack_bf16x2(sc[2 * ks][2], sc[2 * ks][3]);
+                const uint32_t a2 = b2::pack_bf16x2(sc[2 * ks + 1][0], sc[2 * ks + 1][1]),
+                               a3 = b2::pack_bf16x2(sc[2 * ks + 1][2], sc[2 * ks + 1][3]);
+#pragma unroll
+                for (int n2 = 0; n2 < DVT; ++n2) {
+                    uint32_t b0, b1, b2_, b3;
+                    const int key = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), col = n2 * 16 + (lane >> 4) * 8;
+                    b2::ldmatrix_x4_trans(v_base + 2u * (key * LDV + col), b0, b1, b2_, b3);
+                    b2::mma_bf16_16816(o[2 * n2], a0, a1, a2, a3, b0, b1);
+                    b2::mma_bf16_16816(o[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
+                }
             }
         }
-#pragma unroll
-        for (int ks = 0; ks < 4; ++ks) {
-            const uint32_t a0 = b2::pack_bf16x2(sc[2 * ks][0], sc[2 * ks][1]), a1 = b2::pack_bf16x2(sc[2 * ks][2], sc[2 * ks][3]);
-            const uint32_t a2 = b2::pack_bf16x2(sc[2 * ks + 1][0], sc[2 * ks + 1][1]),
-                           a3 = b2::pack_bf16x2(sc[2 * ks + 1][2], sc[2 * ks + 1][3]);
-#pragma unroll
-            for (int n2 = 0; n2 < DVT; ++n2) {
-                uint32_t b0, b1, b2_, b3;
-                const int key = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), col = n2 * 16 + (lane >> 4) * 8;
-                b2::ldmatrix_x4_trans(v_base + 2u * (key * LDV + col), b0, b1, b2_, b3);
-                b2::mma_bf16_16816(o[2 * n2], a0, a1, a2, a3, b0, b1);
-                b2::mma_bf16_16816(o[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
-            }
-        }
+        __syncthreads();                                                    // the tile is consumed: its buffer may be refilled
     }
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
     l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
@@ -705,7 +759,7 @@ int launch_tile(const void* q, const void* k_cache, const void* v_cache, const i
                 int window, int keep_first, float sink, float sink_logit, const float* sink_logits, const float* head_bias,
                 const void* gate, int64_t gate_stride, void* out, int64_t out_stride, cudaStream_t st) {
     constexpr int DK = 16 * DKT, DV = 16 * DVT;
-    const size_t smem = (size_t)(kTQ * (DK + 8) + kTK * (DK + 8) + kTK * (DV + 8)) * sizeof(__nv_bfloat16);
+    const size_t smem = (size_t)(kTQ * (DK + 8) + 2 * kTK * (DK + 8) + 2 * kTK * (DV + 8)) * sizeof(__nv_bfloat16);
     auto kern = chunk_attention_tile_kernel<DKT, DVT, SIG>;
     if (smem > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const int tiles = (T + kTQ - 1) / kTQ + n_seq;          // upper bound on sum(ceil(len / 64)); spare CTAs leave at once

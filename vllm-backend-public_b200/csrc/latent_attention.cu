@@ -805,11 +805,21 @@ window_attention_kernel(const __nv_bfloat16* __restrict__ qn, int64_t qn_row, in
 #pragma unroll
         for (int n = 0; n < 8; ++n) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int j = kv0 + n * 8 + 2 * tq + (e & 1);
-                const bool ok = e < 2 ? (j >= lo0 && j <= i0) : (j >= lo1 && j <= i1);
-                sc[n][e] = ok ? sc[n][e] * scale_log2 : -INFINITY;
+            for (int e = 0; e < 4; ++e) sc[n][e] *= scale_log2;
+        }
+        if (!(kv0 + kWK - 1 <= w_first && (window <= 0 || w_last - kv0 < window))) {       // the warp's rows see the tile in part
+#pragma unroll
+            for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int j = kv0 + n * 8 + 2 * tq + (e & 1);
+                    const bool ok = e < 2 ? (j >= lo0 && j <= i0) : (j >= lo1 && j <= i1);
+                    if (!ok) sc[n][e] = -INFINITY;
+                }
             }
+        }
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
             mx0 = fmaxf(mx0, fmaxf(sc[n][0], sc[n][1]));
             mx1 = fmaxf(mx1, fmaxf(sc[n][2], sc[n][3]));
         }
@@ -819,16 +829,16 @@ window_attention_kernel(const __nv_bfloat16* __restrict__ qn, int64_t qn_row, in
         mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
         const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
         const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
-        const float c0 = exp2f(m0 - mu0), c1 = exp2f(m1 - mu1);
+        const float c0 = b2::fast_exp2(m0 - mu0), c1 = b2::fast_exp2(m1 - mu1);
         m0 = mn0;
         m1 = mn1;
         float s0 = 0.f, s1 = 0.f;
 #pragma unroll
         for (int n = 0; n < 8; ++n) {
-            sc[n][0] = exp2f(sc[n][0] - mu0);
-            sc[n][1] = exp2f(sc[n][1] - mu0);
-            sc[n][2] = exp2f(sc[n][2] - mu1);
-            sc[n][3] = exp2f(sc[n][3] - mu1);
+            sc[n][0] = b2::fast_exp2(sc[n][0] - mu0);
+            sc[n][1] = b2::fast_exp2(sc[n][1] - mu0);
+            sc[n][2] = b2::fast_exp2(sc[n][2] - mu1);
+            sc[n][3] = b2::fast_exp2(sc[n][3] - mu1);
             s0 += sc[n][0] + sc[n][1];
             s1 += sc[n][2] + sc[n][3];
         }
@@ -874,8 +884,8 @@ window_attention_kernel(const __nv_bfloat16* __restrict__ qn, int64_t qn_row, in
     auto gated = [&](const __nv_bfloat16* g, int col, float x, float y) {
         if (gate && gate_channels) {
             const uint32_t z = *reinterpret_cast<const uint32_t*>(g + (size_t)hh * dv + col);
-            x *= b2::sigmoid_f(__uint_as_float(z << 16));
-            y *= b2::sigmoid_f(__uint_as_float(z & 0xffff0000u));
+            x *= b2::sigmoid_as<__nv_bfloat16>(__uint_as_float(z << 16));
+            y *= b2::sigmoid_as<__nv_bfloat16>(__uint_as_float(z & 0xffff0000u));
         }
         return b2::pack_bf16x2(x, y);
     };

@@ -224,6 +224,14 @@ __global__ void gate_mul_kernel(T* __restrict__ out, int64_t out_stride, const T
     }
 }
 
+// W elements per access: 8 (bf16, 16 bytes), 4 (fp32, 16 bytes) or 1.
+template <typename T, int W>
+__device__ __forceinline__ void ld_w(const T* p, float (&v)[W]) {
+    if constexpr (W == 8) b2::ld8(p, v);
+    else if constexpr (W == 4) b2::ld4(p, v);
+    else v[0] = b2::ld(p);
+}
+
 template <typename T, int W>
 __global__ void __launch_bounds__(256)
 parallel_join_kernel(T* __restrict__ out, int64_t out_stride, const T* __restrict__ x, int64_t x_stride, const T* __restrict__ gate,
@@ -233,23 +241,22 @@ parallel_join_kernel(T* __restrict__ out, int64_t out_stride, const T* __restric
     const int first = t < mix_rows ? 0 : n_mix;
     T* o = out + (size_t)t * out_stride;
     for (int i = first + (blockIdx.y * blockDim.x + threadIdx.x) * W; i < n_mix + n_ff; i += gridDim.y * blockDim.x * W) {
-        float v[4] = {0.f, 0.f, 0.f, 0.f}, z[4] = {0.f, 0.f, 0.f, 0.f};
+        float v[W], z[W];
         if (i < n_mix) {
-            const T* xs = x + (size_t)t * x_stride + i;
-            if (W == 4) b2::ld4(xs, v); else v[0] = b2::ld(xs);
+            ld_w<T, W>(x + (size_t)t * x_stride + i, v);
             if (gate) {
-                const T* gs = gate + (size_t)t * gate_stride + i;
-                if (W == 4) b2::ld4(gs, z); else z[0] = b2::ld(gs);
+                ld_w<T, W>(gate + (size_t)t * gate_stride + i, z);
 #pragma unroll
-                for (int c = 0; c < W; ++c) v[c] *= b2::sigmoid_f(z[c]);
+                for (int c = 0; c < W; ++c) v[c] *= b2::sigmoid_as<T>(z[c]);
             }
         } else {
-            const T* us = up + (size_t)t * up_stride + (i - n_mix);
-            if (W == 4) b2::ld4(us, z); else z[0] = b2::ld(us);
+            ld_w<T, W>(up + (size_t)t * up_stride + (i - n_mix), z);
 #pragma unroll
-            for (int c = 0; c < W; ++c) v[c] = act == B2_FF_XIELU ? b2::xielu_f(z[c], a, b) : b2::relu_sq_f(z[c]);
+            for (int c = 0; c < W; ++c) v[c] = act == B2_FF_XIELU ? b2::xielu_as<T>(z[c], a, b) : b2::relu_sq_f(z[c]);
         }
-        if (W == 4) b2::st4(o + i, v); else b2::st(o + i, v[0]);
+        if constexpr (W == 8) b2::st8(o + i, v);
+        else if constexpr (W == 4) b2::st4(o + i, v);
+        else b2::st(o + i, v[0]);
     }
 }
 
@@ -389,22 +396,22 @@ extern "C" int b2_parallel_join(void* out, int64_t out_stride, const void* x, in
     B2_REQUIRE(out && (n_ff == 0 || up) && (mix_rows == 0 || n_mix == 0 || x), B2_EINVAL, "parallel_join: null pointer");
     if (n_ff == 0) T = mix_rows;                                  // nothing to do for the other rows
     cudaStream_t st = static_cast<cudaStream_t>(stream);
-    const size_t esz = act_dtype == B2_ACT_BF16 ? 2 : 4;
-    auto ok = [&](const void* p, int64_t stride) { return !p || (stride % 4 == 0 && reinterpret_cast<uintptr_t>(p) % (4 * esz) == 0); };
-    const bool vec = n_mix % 4 == 0 && n_ff % 4 == 0 && ok(out, out_stride) && ok(x, x_stride) && ok(gate, gate_stride) &&
-                     ok(up, up_stride);
+    const int w = act_dtype == B2_ACT_BF16 ? 8 : 4;
+    auto ok = [&](const void* p, int64_t stride) { return !p || (stride % w == 0 && b2_aligned16(p)); };
+    const bool vec = n_mix % w == 0 && n_ff % w == 0 && ok(out, out_stride) && ok(x, x_stride) && ok(gate, gate_stride) && ok(up, up_stride);
     const int cols = n_mix + n_ff;
-    B2_DISPATCH_ACT(act_dtype, A, {
-        A* o = static_cast<A*>(out);
-        const A* xs = static_cast<const A*>(x);
-        const A* gs = static_cast<const A*>(gate);
-        const A* us = static_cast<const A*>(up);
-        if (vec) parallel_join_kernel<A, 4><<<rows_grid(cols / 4, T), 256, 0, st>>>(o, out_stride, xs, x_stride, gs, gate_stride,
-                                                                                    mix_rows, n_mix, us, up_stride, n_ff, ff_act,
-                                                                                    act_a, act_b);
-        else parallel_join_kernel<A, 1><<<rows_grid(cols, T), 256, 0, st>>>(o, out_stride, xs, x_stride, gs, gate_stride, mix_rows,
-                                                                            n_mix, us, up_stride, n_ff, ff_act, act_a, act_b);
-    });
+#define B2_JOIN(A, W)                                                                                                           \
+    parallel_join_kernel<A, W><<<rows_grid((cols + W - 1) / W, T), 256, 0, st>>>(                                               \
+        static_cast<A*>(out), out_stride, static_cast<const A*>(x), x_stride, static_cast<const A*>(gate), gate_stride, mix_rows, n_mix, \
+        static_cast<const A*>(up), up_stride, n_ff, ff_act, act_a, act_b)
+    if (act_dtype == B2_ACT_BF16) {
+        if (vec) B2_JOIN(__nv_bfloat16, 8);
+        else B2_JOIN(__nv_bfloat16, 1);
+    } else {
+        if (vec) B2_JOIN(float, 4);
+        else B2_JOIN(float, 1);
+    }
+#undef B2_JOIN
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }
