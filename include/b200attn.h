@@ -36,7 +36,7 @@
 extern "C" {
 #endif
 
-#define B2_ABI_VERSION 6
+#define B2_ABI_VERSION 7
 
 #if defined(__GNUC__)
 #define B2_API __attribute__((visibility("default")))
@@ -480,6 +480,12 @@ B2_API int b2_comm_allgather_cols(void* comm, const void* local, int64_t local_s
 #define B2_NORM_RMS   1   /* x / sqrt(mean(x^2) + eps) * w */
 B2_API int b2_embed_streams(float* x, const void* embed, int act_dtype, const int64_t* tokens, int T, int D, int S,
                             float scale, void* stream);
+/* x[t] = embed[token] + bigram[row] in fp32: row = (token before * mul_prev + token * mul_cur) mod buckets, or row `buckets` for
+ * a sequence's first token.  last_token [slots] holds the token before the next portion of every live sequence. */
+B2_API int b2_embed_bigram(float* x, const void* embed, const void* bigram /* [buckets + 1, D] */, int act_dtype,
+                           const int64_t* tokens, int T, int D, int64_t buckets, int64_t mul_prev, int64_t mul_cur,
+                           const int32_t* cu_q, const int32_t* ctx_start, const int32_t* state_slot, int n_seq,
+                           int64_t* last_token, void* stream);
 B2_API int b2_hc_step(float* x, int T, int S, int D, const void* y, int64_t y_stride, const float* mix,
                       const float* out_w, const float* in_w, const float* norm_w, float eps, int norm_kind, void* h,
                       int64_t h_stride, int act_dtype, void* stream);
@@ -504,7 +510,9 @@ B2_API int b2_delta_out(const float* o, const void* proj, int64_t proj_stride, i
 #define B2_GATE_SIGMOID 1
 B2_API int b2_recur_prep(const void* proj, int64_t proj_stride, int act_dtype, int T, int H, int G, int dk, int dv,
                          int taps, const float* conv_w /* NULL with taps = 1: no convolution */, int conv_silu, int unit,
-                         float unit_eps, float q_scale, int off_beta /* < 0: none */, int decay_mode, int off_a,
+                         float unit_eps, float q_scale, float k_scale,
+                         const float* cos_sin /* [max_pos, rot_dims] = cos | sin halves, see b2_qk_rope_cache */, int rot_dims /* 0: q and k
+                         heads are not rotated */, int interleaved, int max_pos, int off_beta /* < 0: none */, int decay_mode, int off_a,
                          const float* a /* fp32 [T, H*dk], channel modes */, int64_t a_stride, const float* A_log,
                          const float* decay_bias /* [H] or [H*dk]; may be NULL in the channel modes */, float tau,
                          const int32_t* cu_q, const int32_t* ctx_start, const int32_t* state_slot, int n_seq,
@@ -514,7 +522,7 @@ B2_API int b2_channel_scan(const float* qkv, const float* beta /* NULL without d
                            const int32_t* ctx_start, const int32_t* state_slot, int n_seq, float* state, float* o,
                            void* stream);
 B2_API int b2_gated_head_norm(const float* o, const void* gate, int64_t gate_stride, int gate_kind, int act_dtype, int T,
-                              int H, int dv, const float* norm_w, float eps, float out_scale, void* out,
+                              int H, int dv, const float* norm_w /* or NULL */, float eps, float out_scale, void* out,
                               int64_t out_stride, void* stream);
 B2_API int b2_qknorm_cache(const void* qkv, int64_t qkv_stride, int act_dtype, int T, int H, int G, int dk, int dv,
                            const float* q_w, const float* k_w, float eps, const int64_t* slots, int bs, void* q_out,
@@ -531,14 +539,18 @@ B2_API int b2_chunk_attention(void* out, const void* q, const void* k_cache, con
  * (position i sees j <= i with i - j < window or j < keep_first; window = 0: none), the sink's logit per query head
  * (sink_logits [H] fp32, or NULL: sink_logit for all), a sigmoid gate per (token, head) on the output (gate rows of the
  * activation type with gate_stride elements between tokens, or NULL), the kind of a key's weight, and output rows
- * [H * dv] with out_stride elements between tokens.  B2_WEIGHT_SIGMOID takes head_bias [H] fp32 (or NULL: 0) and no sink. */
+ * [H * dv] with out_stride elements between tokens.  B2_WEIGHT_SIGMOID takes head_bias [H] fp32 (or NULL: 0) and no sink.
+ * softcap > 0: scores become softcap * tanh(score / softcap).  maps = 2: q is [T, H, 2, dk] and the K pool [nb, G * 2, bs, dk];
+ * each of a head's two maps is a softmax attention of its own over the values, and the head's output is
+ * d / sqrt(mean(d^2) + map_eps) * map_scale with d = a1 - map_lambda * a2 (map_lambda, map_eps, map_scale unused with maps = 1). */
 #define B2_WEIGHT_SOFTMAX 0       /* exp(s_j) / (sink + sum exp(s)) */
 #define B2_WEIGHT_SIGMOID 1       /* sigmoid(s_j + head_bias[h]), not normalised over the keys */
 B2_API int b2_masked_attention(void* out, const void* q, const void* k_cache, const void* v_cache, int act_dtype,
                                const int32_t* block_tables, int max_nb, const int32_t* cu_q, const int32_t* ctx_start,
                                int n_seq, int T, int H, int G, int dk, int dv, int bs, float scale, int chunk, int window,
                                int keep_first, float sink, float sink_logit, const float* sink_logits, int weight_kind,
-                               const float* head_bias, const void* gate, int64_t gate_stride, int64_t out_stride, void* stream);
+                               const float* head_bias, const void* gate, int64_t gate_stride, float softcap, int maps,
+                               float map_lambda, float map_eps, float map_scale, int64_t out_stride, void* stream);
 /* rows [q (H*dk) | k (G*dk)] or [q | k | v (G*dv)]: the first rot_dims entries of every q and k head turn by the token's
  * position (pairs (i, i + rot_dims/2), or (2i, 2i+1) when interleaved; cos_sin fp32 [max_pos, rot_dims] = cos | sin
  * halves), q -> q_out [T, H, dk], rotated k -> K pool; the V pool gets v, or with v_from_k the k heads BEFORE the rotation. */
@@ -547,8 +559,8 @@ B2_API int b2_qk_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, 
                             int max_pos, const int64_t* slots, int bs, void* q_out, void* k_cache, void* v_cache,
                             void* stream);
 /* the same after an RMS norm over all of q (H*dk numbers, weight q_w) and over all of k (G*dk, weight k_w); both weights NULL:
- * no norm */
-B2_API int b2_qk_norm_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, int T, int H, int G, int dk, int dv,
+ * no norm.  Gv <= G value heads: v has Gv * dv numbers and the V pool Gv heads (several key maps over one set of values) */
+B2_API int b2_qk_norm_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, int T, int H, int G, int Gv, int dk, int dv,
                                  int v_from_k, const float* q_w, const float* k_w, float eps, int rot_dims, int interleaved,
                                  const int32_t* positions, const float* cos_sin, int max_pos, const int64_t* slots, int bs,
                                  void* q_out, void* k_cache, void* v_cache, void* stream);
@@ -558,6 +570,7 @@ B2_API int b2_moe_capacity(int n, int E);
 #define B2_ROUTE_SOFTMAX_ALL  1   /* s = softmax over all experts, top-k of s + bias, weights = the chosen s as they are */
 #define B2_ROUTE_SIGMOID_GROUPED 2 /* s = sigmoid, choice by s + bias inside the keep_groups best of n_groups groups (group score =
                                    * its two largest s + bias), weights = chosen s / (their sum + 1e-20) * weight_scale */
+#define B2_ROUTE_SIGMOID_PLAIN 3  /* the same choice, weights = chosen s * weight_scale, not divided by their sum */
 #define B2_GLU_SILU    0          /* silu(g) * u */
 #define B2_GLU_CLAMPED 1          /* g' = min(g, limit), u' = clamp(u, -limit, limit): g' * sigmoid(alpha g') * (u' + 1) */
 #define B2_GLU_GELU_TANH 2        /* gelu_tanh(g) * u (b2_glu_and_mul only) */
@@ -573,19 +586,28 @@ B2_API int b2_moe_select_ex(const float* logits, int64_t stride, const float* bi
                             int n_groups, int keep_groups, float weight_scale, int32_t* ids, float* weights, void* stream);
 B2_API int b2_moe_align(const int32_t* ids, int n, int E, int cap, int32_t* sorted, int32_t* tile_expert, int32_t* place,
                         int32_t* group_ends /* [E] or NULL */, void* stream);
-B2_API int b2_moe_gather(const void* h, int64_t h_stride, int act_dtype, const int32_t* sorted, int cap, int top, int D,
-                         void* out, void* stream);
-B2_API int b2_moe_combine(const void* rows, int rows_f32, const int32_t* place, const float* weights, int T, int top, int D,
-                          void* y, int64_t y_stride, int act_dtype, void* stream);
+B2_API int b2_moe_gather(const void* h, int64_t h_stride, int act_dtype, const int32_t* sorted,
+                         const float* weights /* [T, top]: scales the rows, or NULL */, int cap, int top, int D, void* out,
+                         void* stream);
+B2_API int b2_moe_combine(const void* rows, int rows_f32, const int32_t* place, const float* weights /* NULL: ones */, int T,
+                          int top, int D, const void* add /* rows joining the sum, or NULL */, int64_t add_stride, void* y,
+                          int64_t y_stride, int act_dtype, void* stream);
 B2_API int b2_moe_experts(const void* h, int64_t h_stride, const void* w_gate, const void* w_up, const void* w_down,
                           int64_t w13_expert_stride /* elements between experts of w_gate / w_up (>= F*D) */,
                           int act_dtype, int T, int D, int F, int top, int cap, const int32_t* sorted,
                           const int32_t* tile_expert, const int32_t* place, const float* weights, void* act, float* rows,
-                          void* y, int64_t y_stride, int glu, float glu_alpha, float glu_limit, void* stream);
+                          const void* add /* rows joining the sum (a shared expert's output), or NULL */, int64_t add_stride,
+                          void* y, int64_t y_stride, int glu, float glu_alpha, float glu_limit,
+                          int weight_on_input /* 1: sum of expert(weight * h) instead of weight * expert(h) */, void* stream);
 /* post_norm.cu: norms on both sides of a sublayer around an fp32 residual, element-wise activations, logit soft cap */
 B2_API int b2_sandwich_norm(float* x, int T, int D, const void* y, int64_t y_stride, const float* post_w,
                             const float* post_b, const float* pre_w, const float* pre_b, float eps, int norm_kind, void* h,
                             int64_t h_stride, int act_dtype, void* stream);
+/* RMS norms around a sublayer output in two halves: y = pair_scale * (norm(y1; w1) + norm(y2; w2)), x <- x + norm(y; post_w)
+ * (post_w NULL: x + y), h = norm(x; pre_w) when given */
+B2_API int b2_sandwich_norm_pair(float* x, int T, int D, const void* y1, int64_t y1_stride, const float* w1, const void* y2,
+                                 int64_t y2_stride, const float* w2, float pair_scale, const float* post_w, const float* pre_w,
+                                 float eps, void* h, int64_t h_stride, int act_dtype, void* stream);
 B2_API int b2_row_norm(void* out, int64_t out_stride, const void* in, int64_t in_stride, int act_dtype, int T, int n,
                        const float* w /* [n] or NULL */, float eps, void* stream);
 B2_API int b2_relu_sq(void* out, int64_t out_stride, const void* in, int64_t in_stride, int act_dtype, int T, int I,

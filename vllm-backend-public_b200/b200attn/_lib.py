@@ -20,10 +20,10 @@ CORE_LIB_PATH = PKG_ROOT / "lib" / "libb200core.so"
 
 B2_OK, B2_EINVAL, B2_EUNSUPPORTED, B2_ECUDA, B2_ENOMEM, B2_ENOTFOUND, B2_EEXISTS = 0, -1, -2, -3, -4, -5, -6
 KV_BF16, KV_FP8_E4M3 = 0, 1
-ABI_VERSION = 6
+ABI_VERSION = 7
 ACT_BF16, ACT_F32 = 0, 1
 NORM_LAYER, NORM_RMS = 0, 1
-ROUTE_TOPK_SOFTMAX, ROUTE_SOFTMAX_ALL, ROUTE_SIGMOID_GROUPED = 0, 1, 2
+ROUTE_TOPK_SOFTMAX, ROUTE_SOFTMAX_ALL, ROUTE_SIGMOID_GROUPED, ROUTE_SIGMOID_PLAIN = 0, 1, 2, 3
 GLU_SILU, GLU_CLAMPED, GLU_GELU_TANH, FF_RELU_SQ, FF_XIELU = 0, 1, 2, 3, 4
 WEIGHT_SOFTMAX, WEIGHT_SIGMOID = 0, 1
 DECAY_HEAD_SOFTPLUS, DECAY_CHANNEL_SOFTPLUS, DECAY_CHANNEL_SIGMOID_POW, DECAY_HEAD_CONST = 0, 1, 2, 3
@@ -109,13 +109,14 @@ SIGNATURES = {
     "b2_comm_push_allreduce_rms_norm": (i32, [vp, vp, i64, vp, vp, vp, i32, i64, i64, f32, vp]),
     "b2_comm_allgather_cols": (i32, [vp, vp, i64, i32, i32, vp]),
     "b2_embed_streams": (i32, [vp, vp, i32, vp, i32, i32, i32, f32, vp]),
+    "b2_embed_bigram": (i32, [vp, vp, vp, i32, vp, i32, i32, i64, i64, i64, vp, vp, vp, i32, vp, vp]),
     "b2_hc_step": (i32, [vp, i32, i32, i32, vp, i64, vp, vp, vp, vp, f32, i32, vp, i64, i32, vp]),
     "b2_delta_prep": (i32, [vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp,
                             vp, vp]),
     "b2_delta_scan": (i32, [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, vp, i32, vp, vp, vp]),
     "b2_delta_out": (i32, [vp, vp, i64, i32, i32, i32, i32, i32, vp, f32, vp, i64, vp]),
-    "b2_recur_prep": (i32, [vp, i64, i32, i32, i32, i32, i32, i32, i32, vp, i32, i32, f32, f32, i32, i32, i32, vp, i64, vp, vp, f32,
-                            vp, vp, vp, i32, vp, vp, vp, vp, vp]),
+    "b2_recur_prep": (i32, [vp, i64, i32, i32, i32, i32, i32, i32, i32, vp, i32, i32, f32, f32, f32, vp, i32, i32, i32, i32, i32, i32,
+                            vp, i64, vp, vp, f32, vp, vp, vp, i32, vp, vp, vp, vp, vp]),
     "b2_channel_scan": (i32, [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp, i32, vp, vp, vp]),
     "b2_gated_head_norm": (i32, [vp, vp, i64, i32, i32, i32, i32, i32, vp, f32, f32, vp, i64, vp]),
     "b2_qk_prep_cache": (i32, [vp, i64, i32, i32, i32, i32, i32, i32, i32, vp, vp, f32, vp, f32, i32, vp, i32, vp, vp, vp, vp]),
@@ -123,9 +124,9 @@ SIGNATURES = {
     "b2_chunk_attention": (i32, [vp, vp, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, f32,
                                  f32, vp]),
     "b2_masked_attention": (i32, [vp, vp, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32,
-                                  f32, f32, vp, i32, vp, vp, i64, i64, vp]),
+                                  f32, f32, vp, i32, vp, vp, i64, f32, i32, f32, f32, f32, i64, vp]),
     "b2_qk_rope_cache": (i32, [vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp, i32, vp, vp, vp, vp]),
-    "b2_qk_norm_rope_cache": (i32, [vp, i64, i32, i32, i32, i32, i32, i32, i32, vp, vp, f32, i32, i32, vp, vp, i32, vp, i32, vp, vp,
+    "b2_qk_norm_rope_cache": (i32, [vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, f32, i32, i32, vp, vp, i32, vp, i32, vp, vp,
                                     vp, vp]),
     "b2_moe_tile_rows": (i32, []),
     "b2_moe_capacity": (i32, [i32, i32]),
@@ -134,11 +135,12 @@ SIGNATURES = {
     "b2_moe_route_ex": (i32, [vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp]),
     "b2_moe_select_ex": (i32, [vp, i64, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp]),
     "b2_moe_align": (i32, [vp, i32, i32, i32, vp, vp, vp, vp, vp]),
-    "b2_moe_gather": (i32, [vp, i64, i32, vp, i32, i32, i32, vp, vp]),
-    "b2_moe_combine": (i32, [vp, i32, vp, vp, i32, i32, i32, vp, i64, i32, vp]),
-    "b2_moe_experts": (i32, [vp, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, i64, i32, f32,
-                             f32, vp]),
+    "b2_moe_gather": (i32, [vp, i64, i32, vp, vp, i32, i32, i32, vp, vp]),
+    "b2_moe_combine": (i32, [vp, i32, vp, vp, i32, i32, i32, vp, i64, vp, i64, i32, vp]),
+    "b2_moe_experts": (i32, [vp, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, i64, vp, i64, i32,
+                             f32, f32, i32, vp]),
     "b2_sandwich_norm": (i32, [vp, i32, i32, vp, i64, vp, vp, vp, vp, f32, i32, vp, i64, i32, vp]),
+    "b2_sandwich_norm_pair": (i32, [vp, i32, i32, vp, i64, vp, vp, i64, vp, f32, vp, vp, f32, vp, i64, i32, vp]),
     "b2_row_norm": (i32, [vp, i64, vp, i64, i32, i32, i32, vp, f32, vp]),
     "b2_relu_sq": (i32, [vp, i64, vp, i64, i32, i32, i32, vp]),
     "b2_glu_and_mul": (i32, [vp, i64, vp, i64, i32, i32, i32, i32, f32, f32, vp]),

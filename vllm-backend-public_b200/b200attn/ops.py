@@ -644,7 +644,7 @@ from dataclasses import dataclass  # noqa: E402
 
 from ._lib import (ACT_BF16, ACT_F32, DECAY_CHANNEL_SIGMOID_POW, DECAY_CHANNEL_SOFTPLUS,  # noqa: E402,F401
                    DECAY_HEAD_CONST, DECAY_HEAD_SOFTPLUS, FF_RELU_SQ, FF_XIELU, GATE_SIGMOID, GATE_SILU, GLU_CLAMPED, GLU_GELU_TANH, GLU_SILU, NORM_LAYER,
-                   NORM_RMS, ROUTE_SIGMOID_GROUPED, ROUTE_SOFTMAX_ALL, ROUTE_TOPK_SOFTMAX, WEIGHT_SIGMOID, WEIGHT_SOFTMAX)
+                   NORM_RMS, ROUTE_SIGMOID_GROUPED, ROUTE_SIGMOID_PLAIN, ROUTE_SOFTMAX_ALL, ROUTE_TOPK_SOFTMAX, WEIGHT_SIGMOID, WEIGHT_SOFTMAX)
 
 
 def _act(t: torch.Tensor, name: str) -> int:
@@ -714,6 +714,26 @@ def embed_streams(embed: torch.Tensor, tokens: torch.Tensor, streams: int, scale
     x = torch.empty(T, streams, D, dtype=torch.float32, device=dev)
     _lib.check(lib.b2_embed_streams(_ptr(x), _ptr(embed), _act(embed, "embed"), _ptr(tokens), T, D, streams, float(scale),
                                     _stream(dev)))
+    return x
+
+
+def embed_bigram(embed: torch.Tensor, bigram: torch.Tensor, tokens: torch.Tensor, batch: SeqBatch, mul_prev: int, mul_cur: int,
+                 last_token: torch.Tensor) -> torch.Tensor:
+    """x[t] = embed[token] + bigram[(token before * mul_prev + token * mul_cur) mod buckets] as fp32 [T, D]; bigram
+    [buckets + 1, D], its last row for a sequence's first token.  last_token int64 [slots]: the token before the next portion of
+    every live sequence, read for a portion's first row and advanced to its last token.  b2_embed_bigram."""
+    lib = _lib.load()
+    dev = _need_cuda(embed=embed, bigram=bigram, tokens=tokens, last_token=last_token)
+    if tokens.dtype != torch.int64 or not tokens.is_contiguous() or not embed.is_contiguous() or not bigram.is_contiguous() \
+            or bigram.dtype != embed.dtype or bigram.shape[1] != embed.shape[1]:
+        raise ValueError("tokens must be contiguous int64, embed and bigram contiguous, of one width and dtype")
+    if last_token.dtype != torch.int64 or not last_token.is_contiguous() or batch.state_slots is None:
+        raise ValueError("last_token must be contiguous int64 [slots], and the batch must carry its state slots")
+    T, D = tokens.shape[0], embed.shape[1]
+    x = torch.empty(T, D, dtype=torch.float32, device=dev)
+    _lib.check(lib.b2_embed_bigram(_ptr(x), _ptr(embed), _ptr(bigram), _act(embed, "embed"), _ptr(tokens), T, D, bigram.shape[0] - 1,
+                                   int(mul_prev), int(mul_cur), _ptr(batch.cu_q), _ptr(batch.ctx_start), _ptr(batch.state_slots),
+                                   batch.n_seq, _ptr(last_token), _stream(dev)))
     return x
 
 
@@ -834,19 +854,24 @@ def chunk_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     chunk: int = 0, sink: float = 0.0, sink_logit: float = 0.0, window: int = 0, keep_first: int = 0,
                     sink_logits: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                     weight_kind: int = WEIGHT_SOFTMAX, head_bias: Optional[torch.Tensor] = None,
-                    out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    out: Optional[torch.Tensor] = None, softcap: float = 0.0, maps: int = 1, map_lambda: float = 0.0,
+                    map_eps: float = 1e-6, map_scale: float = 1.0) -> torch.Tensor:
     """Attention of q [T, H, dk] over the paged pools.  Row at position p sees positions j <= p with
     j // chunk == p // chunk (chunk = 0: all j <= p) and, with a window > 0, p - j < window or j < keep_first; the
     denominator carries sink * exp(sink_logit), or sink * exp(sink_logits[h]) with one fp32 logit per query head; with
     gate [T, H] (q's dtype, a column slice of a wider row is fine) head h's output is multiplied by sigmoid(gate[t, h]).
     weight_kind WEIGHT_SIGMOID: a visible key weighs sigmoid(score + head_bias[h]) (fp32 [H] or None), not normalised; no sink.
+    softcap > 0: scores become softcap * tanh(score / softcap).  maps = 2 (differential attention): q [T, 2 H, dk], two maps per
+    head side by side, k_cache [nb, 2 G, bs, dk]; head h gives d / sqrt(mean(d^2) + map_eps) * map_scale, d = a1 - map_lambda * a2.
     Returns [T, H, dv] of q's dtype, or `out`: rows [T, >= H * dv] (a column range of a wider buffer).  b2_masked_attention."""
     lib = _lib.load()
     dev = _need_cuda(q=q, k_cache=k_cache, v_cache=v_cache, sink_logits=sink_logits, gate=gate, head_bias=head_bias, out=out)
     T, H, dk = q.shape
     nb, G, bs, dv = v_cache.shape
-    if not q.is_contiguous() or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype or tuple(k_cache.shape) != (nb, G, bs, dk):
-        raise ValueError("q must be contiguous and the pools of its dtype, k_cache [nb, G, bs, dk]")
+    if maps < 1 or H % maps or not q.is_contiguous() or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype \
+            or tuple(k_cache.shape) != (nb, G * maps, bs, dk):
+        raise ValueError("q must be contiguous and the pools of its dtype, k_cache [nb, maps * G, bs, dk]")
+    H //= maps
     bt = batch.block_tables
     if bt is None or bt.dtype != torch.int32 or bt.dim() != 2 or bt.stride(1) != 1 or bt.shape[0] < batch.n_seq \
             or (bt.shape[0] > 1 and bt.stride(0) != bt.shape[1]):
@@ -864,7 +889,8 @@ def chunk_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     _lib.check(lib.b2_masked_attention(_ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), _act(q, "q"), _ptr(bt), bt.shape[1],
                                        _ptr(batch.cu_q), _ptr(batch.ctx_start), batch.n_seq, T, H, G, dk, dv, bs,
                                        float(scale), int(chunk), int(window), int(keep_first), float(sink), float(sink_logit),
-                                       _ptr(sink_logits), int(weight_kind), _ptr(head_bias), _ptr(gate), gs, os_, _stream(dev)))
+                                       _ptr(sink_logits), int(weight_kind), _ptr(head_bias), _ptr(gate), gs, float(softcap), int(maps),
+                                       float(map_lambda), float(map_eps), float(map_scale), os_, _stream(dev)))
     return out
 
 
@@ -872,22 +898,22 @@ def qk_rope_cache(qkv: torch.Tensor, H: int, G: int, dk: int, dv: int, positions
                   rot_dims: int, slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, interleaved: bool = False,
                   v_from_k: bool = False, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None,
                   eps: float = 1e-6) -> torch.Tensor:
-    """Rows qkv [T, >= H*dk + G*dk (+ G*dv)] = q | k (| v), biases already added: the first rot_dims entries of every q and k
+    """Rows qkv [T, >= H*dk + G*dk (+ Gv*dv)] = q | k (| v), biases already added: the first rot_dims entries of every q and k
     head turn by the token's position (pairs (i, i + rot_dims/2), interleaved: (2i, 2i + 1); cos_sin from rotary_table),
     rotated k goes to k_cache [nb, G, bs, dk] and v -- with v_from_k the k heads as projected, before the rotation -- to
-    v_cache [nb, G, bs, dv] at slots[t] (< 0 skips).  q_norm [H*dk] / k_norm [G*dk] (fp32, both or none): all of q and all of k
+    v_cache [nb, Gv, bs, dv] at slots[t] (< 0 skips); Gv = G, or fewer value heads than key heads.  q_norm [H*dk] / k_norm [G*dk] (fp32, both or none): all of q and all of k
     are RMS-normed as one row each before that.  Returns the rotated q [T, H, dk].  b2_qk_norm_rope_cache."""
     lib = _lib.load()
     _f32(q_norm, "q_norm", (H * dk,)), _f32(k_norm, "k_norm", (G * dk,))
     _need_cuda(q_norm=q_norm, k_norm=k_norm)
     dev = _need_cuda(qkv=qkv, slots=slots, k_cache=k_cache, v_cache=v_cache, positions=positions, cos_sin=cos_sin)
     T, P, ps = _mat(qkv, "qkv")
-    if P < H * dk + G * dk + (0 if v_from_k else G * dv):
+    nb, bs, Gv = k_cache.shape[0], k_cache.shape[2], v_cache.shape[1]
+    if P < H * dk + G * dk + (0 if v_from_k else Gv * dv):
         raise ValueError("qkv is narrower than its heads")
-    nb, bs = k_cache.shape[0], k_cache.shape[2]
-    if tuple(k_cache.shape) != (nb, G, bs, dk) or tuple(v_cache.shape) != (nb, G, bs, dv) or not k_cache.is_contiguous() \
+    if tuple(k_cache.shape) != (nb, G, bs, dk) or tuple(v_cache.shape) != (nb, Gv, bs, dv) or Gv > G or not k_cache.is_contiguous() \
             or not v_cache.is_contiguous() or k_cache.dtype != qkv.dtype or v_cache.dtype != qkv.dtype:
-        raise ValueError("k_cache / v_cache must be contiguous [nb, G, bs, dk] / [nb, G, bs, dv] of qkv's dtype")
+        raise ValueError("k_cache / v_cache must be contiguous [nb, G, bs, dk] / [nb, Gv, bs, dv] of qkv's dtype")
     if slots.dtype != torch.int64 or slots.shape != (T,) or not slots.is_contiguous():
         raise ValueError("slots must be contiguous int64 [T]")
     if positions.dtype != torch.int32 or positions.shape != (T,) or not positions.is_contiguous():
@@ -896,7 +922,7 @@ def qk_rope_cache(qkv: torch.Tensor, H: int, G: int, dk: int, dv: int, positions
                      or not cos_sin.is_contiguous()):
         raise ValueError(f"cos_sin must be contiguous fp32 [max_pos, {rot_dims}]")
     q = torch.empty(T, H, dk, dtype=qkv.dtype, device=dev)
-    _lib.check(lib.b2_qk_norm_rope_cache(_ptr(qkv), ps, _act(qkv, "qkv"), T, H, G, dk, dv, int(v_from_k), _ptr(q_norm), _ptr(k_norm),
+    _lib.check(lib.b2_qk_norm_rope_cache(_ptr(qkv), ps, _act(qkv, "qkv"), T, H, G, Gv, dk, dv, int(v_from_k), _ptr(q_norm), _ptr(k_norm),
                                          float(eps), int(rot_dims), int(interleaved), _ptr(positions), _ptr(cos_sin),
                                          cos_sin.shape[0] if rot_dims else 1, _ptr(slots), bs, _ptr(q), _ptr(k_cache),
                                          _ptr(v_cache), _stream(dev)))
@@ -909,7 +935,7 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tens
     weights = softmax over the chosen; ROUTE_SOFTMAX_ALL: s = softmax(z) over all experts, the top s + bias are chosen,
     weights = their s, not renormalised; ROUTE_SIGMOID_GROUPED: s = sigmoid(z), the top s + bias inside the `keep_groups`
     of `n_groups` groups of neighbouring experts with the largest sum of their two best s + bias, weights = the chosen s
-    over their sum, times weight_scale."""
+    over their sum, times weight_scale; ROUTE_SIGMOID_PLAIN: the same choice, weights = the chosen s * weight_scale."""
     lib = _lib.load()
     dev = _need_cuda(h=h, w_router=w_router, bias=bias)
     T, D, hs = _mat(h, "h")
@@ -942,10 +968,13 @@ MOE_GROUPED_GEMM_MIN_PAIRS = 2048
 
 def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate: Optional[torch.Tensor], w_up: torch.Tensor,
                 w_down: torch.Tensor, w_gate_up: Optional[torch.Tensor] = None, glu: int = GLU_SILU,
-                glu_alpha: float = 1.0, glu_limit: float = 0.0) -> torch.Tensor:
+                glu_alpha: float = 1.0, glu_limit: float = 0.0, weight_on_input: bool = False,
+                add: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y[t] = sum_j wts[t, j] * W_down[e] glu(W_gate[e] h[t], W_up[e] h[t]), e = ids[t, j]; glu = silu(g) * u (GLU_SILU) or
     the bounded unit min(g, limit) * sigmoid(alpha min(g, limit)) * (clamp(u, +-limit) + 1) (GLU_CLAMPED); FF_RELU_SQ:
     experts without a gate, y[t] = sum_j wts[t, j] * W_down[e] max(W_up[e] h[t], 0)^2 (w_gate None).
+    weight_on_input: y[t] = sum_j expert_e(wts[t, j] * h[t]) instead; add [T, D] (h's dtype): joins the sum in fp32 (the output of
+    an expert that every token uses).
     w_gate, w_up [E, F, D]; w_down [E, D, F]; w_gate_up [E, 2F, D] (optional): the two stacked per expert -- w_gate and
     w_up may be views of it.  Sorting by expert (b2_moe_align), both products and the weighted sum (in fp32, choice order)
     run on the device without a host read: b2_moe_experts, or for large bf16 batches b2_moe_gather -> grouped GEMM ->
@@ -966,6 +995,12 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate: O
     if ids.dtype != torch.int32 or not ids.is_contiguous() or tuple(ids.shape) != (T, top):
         raise ValueError("ids must be contiguous int32 [T, top]")
     _f32(wts, "wts", (T, top))
+    as_ = 0
+    if add is not None:
+        Ta, Da, as_ = _mat(add, "add")
+        if (Ta, Da) != (T, D) or add.dtype != h.dtype:
+            raise ValueError("add must be [T, D] of h's dtype")
+        _need_cuda(add=add)
     n = T * top
     cap = lib.b2_moe_capacity(n, E)
     tiles = cap // lib.b2_moe_tile_rows()
@@ -982,20 +1017,22 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gate: O
         if tuple(w_gate_up.shape) != (E, (2 if gated else 1) * F, D) or not w_gate_up.is_contiguous() or w_gate_up.dtype != h.dtype:
             raise ValueError("w_gate_up must be contiguous [E, 2F, D] of h's dtype")
         a = torch.empty(cap, D, dtype=h.dtype, device=dev)
-        _lib.check(lib.b2_moe_gather(_ptr(h), hs, _act(h, "h"), _ptr(srt), cap, top, D, _ptr(a), _stream(dev)))
+        _lib.check(lib.b2_moe_gather(_ptr(h), hs, _act(h, "h"), _ptr(srt), _ptr(wts) if weight_on_input else None, cap, top, D,
+                                     _ptr(a), _stream(dev)))
         gu = torch._grouped_mm(a, w_gate_up.transpose(1, 2), offs=ends)              # [cap, 2F]; rows past the last group unset
         if not gated:
             act = relu_sq(gu)
         else:
             act = silu_and_mul(gu) if glu == GLU_SILU else glu_and_mul(gu, glu, glu_alpha, glu_limit)
         rows = torch._grouped_mm(act, w_down.transpose(1, 2), offs=ends)             # [cap, D]
-        _lib.check(lib.b2_moe_combine(_ptr(rows), 0, _ptr(place), _ptr(wts), T, top, D, _ptr(y), D, _act(h, "h"), _stream(dev)))
+        _lib.check(lib.b2_moe_combine(_ptr(rows), 0, _ptr(place), None if weight_on_input else _ptr(wts), T, top, D, _ptr(add), as_,
+                                      _ptr(y), D, _act(h, "h"), _stream(dev)))
         return y
     act = torch.empty(cap, F, dtype=h.dtype, device=dev)
     rows = torch.empty(cap, D, dtype=torch.float32, device=dev)
     _lib.check(lib.b2_moe_experts(_ptr(h), hs, _ptr(w_gate), _ptr(w_up), _ptr(w_down), w_up.stride(0), _act(h, "h"), T, D, F,
-                                  top, cap, _ptr(srt), _ptr(tile_e), _ptr(place), _ptr(wts), _ptr(act), _ptr(rows), _ptr(y), D,
-                                  int(glu), float(glu_alpha), float(glu_limit), _stream(dev)))
+                                  top, cap, _ptr(srt), _ptr(tile_e), _ptr(place), _ptr(wts), _ptr(act), _ptr(rows), _ptr(add), as_,
+                                  _ptr(y), D, int(glu), float(glu_alpha), float(glu_limit), int(weight_on_input), _stream(dev)))
     return y
 
 
@@ -1089,10 +1126,13 @@ def recur_prep(proj: torch.Tensor, H: int, G: int, dk: int, dv: int, batch: SeqB
                conv_w: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None, conv_silu: bool = False,
                unit: bool = False, unit_eps: float = 1e-6, q_scale: float = 1.0, off_beta: int = -1,
                decay_mode: int = DECAY_CHANNEL_SOFTPLUS, off_a: int = -1, a: Optional[torch.Tensor] = None,
-               A_log: Optional[torch.Tensor] = None, decay_bias: Optional[torch.Tensor] = None, tau: float = 1.0):
+               A_log: Optional[torch.Tensor] = None, decay_bias: Optional[torch.Tensor] = None, tau: float = 1.0,
+               k_scale: float = 1.0, cos_sin: Optional[torch.Tensor] = None, interleaved: bool = False):
     """Inputs of a linear recurrence over a matrix state from projection rows proj [T, >= 2*G*dk + H*dv] whose first columns
     are q | k | v: optional short causal convolution (taps, conv_w [C, taps], tail in conv_state [slots, taps-1, C]) with
-    optional SiLU, optional unit vectors for the q and k heads (x / sqrt(sum x^2 + unit_eps)), q times q_scale,
+    optional SiLU, optional unit vectors for the q and k heads (x / sqrt(sum x^2 + unit_eps)), q times q_scale, k times k_scale,
+    with cos_sin (fp32 [max_pos, rot_dims] from rotary_table) the first rot_dims entries of every q and k head rotated by the
+    token's position (pairs (i, i + rot_dims/2), interleaved: (2i, 2i + 1)),
     beta = sigmoid(proj[:, off_beta + h]) when off_beta >= 0, and the decay: DECAY_HEAD_SOFTPLUS [T, H] from proj[:, off_a + h],
     A_log [H], decay_bias [H]; DECAY_CHANNEL_SOFTPLUS [T, H, dk] = exp(-exp(A_log[h]) softplus(a + decay_bias));
     DECAY_CHANNEL_SIGMOID_POW [T, H, dk] = sigmoid(a + decay_bias)^(1 / tau), a fp32 [T, H*dk]; DECAY_HEAD_CONST [T, H] =
@@ -1125,11 +1165,18 @@ def recur_prep(proj: torch.Tensor, H: int, G: int, dk: int, dv: int, batch: SeqB
     _f32(A_log, "A_log", (H,))
     if batch.state_slots is None:
         raise ValueError("the batch carries no state slots")
+    rot_dims, max_pos = 0, 1
+    if cos_sin is not None:
+        if cos_sin.dtype != torch.float32 or cos_sin.dim() != 2 or not cos_sin.is_contiguous():
+            raise ValueError("cos_sin must be contiguous fp32 [max_pos, rot_dims]")
+        max_pos, rot_dims = cos_sin.shape
+        _need_cuda(cos_sin=cos_sin)
     qkv = torch.empty(T, C, dtype=torch.float32, device=dev)
     beta = torch.empty(T, H, dtype=torch.float32, device=dev) if off_beta >= 0 else None
     decay = torch.empty(T, H * (dk if per_channel else 1), dtype=torch.float32, device=dev)
     _lib.check(lib.b2_recur_prep(_ptr(proj), ps, _act(proj, "proj"), T, H, G, dk, dv, int(taps), _ptr(conv_w), int(conv_silu),
-                                 int(unit), float(unit_eps), float(q_scale), int(off_beta), int(decay_mode), int(off_a), _ptr(a),
+                                 int(unit), float(unit_eps), float(q_scale), float(k_scale), _ptr(cos_sin) if rot_dims else None, rot_dims,
+                                 int(interleaved), max_pos, int(off_beta), int(decay_mode), int(off_a), _ptr(a),
                                  a_stride, _ptr(A_log), _ptr(decay_bias), float(tau), _ptr(batch.cu_q), _ptr(batch.ctx_start),
                                  _ptr(batch.state_slots), batch.n_seq, _ptr(conv_state), _ptr(qkv), _ptr(beta), _ptr(decay),
                                  _stream(dev)))
@@ -1159,10 +1206,10 @@ def channel_scan(qkv: torch.Tensor, beta: Optional[torch.Tensor], decay: torch.T
     return o
 
 
-def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, norm_w: torch.Tensor, eps: float, gate_kind: int = GATE_SILU,
+def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, norm_w: Optional[torch.Tensor], eps: float, gate_kind: int = GATE_SILU,
                     out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """o fp32 [T, H, dv] -> o / rms(o over dv) * norm_w * act(gate) * out_scale as [T, H*dv] of gate's dtype; gate [T, H*dv]
-    (a view with a row stride is fine), act = SiLU or sigmoid.  b2_gated_head_norm."""
+    """o fp32 [T, H, dv] -> o / rms(o over dv) * norm_w * act(gate) * out_scale as [T, H*dv] of gate's dtype (norm_w None: no
+    weight); gate [T, H*dv] (a view with a row stride is fine), act = SiLU or sigmoid.  b2_gated_head_norm."""
     lib = _lib.load()
     dev = _need_cuda(o=o, gate=gate, norm_w=norm_w, out=out)
     T, H, dv = o.shape
@@ -1291,6 +1338,27 @@ def sandwich_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, post_w: Opt
     return h
 
 
+def sandwich_norm_pair(x: torch.Tensor, y1: torch.Tensor, w1: torch.Tensor, y2: torch.Tensor, w2: torch.Tensor, pair_scale: float,
+                       post_w: Optional[torch.Tensor], pre_w: Optional[torch.Tensor] = None, eps: float = 1e-6) -> Optional[torch.Tensor]:
+    """sandwich_norm (RMS) with a sublayer output in two halves: y = pair_scale * (rms(y1) * w1 + rms(y2) * w2), all in fp32;
+    x <- x + rms(y) * post_w (post_w None: x + y); with pre_w returns h = rms(x) * pre_w as y1's dtype.  b2_sandwich_norm_pair."""
+    lib = _lib.load()
+    dev = _need_cuda(x=x, y1=y1, w1=w1, y2=y2, w2=w2, post_w=post_w, pre_w=pre_w)
+    if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous():
+        raise ValueError("x must be contiguous fp32 [T, D]")
+    T, D = x.shape
+    T1, D1, s1 = _mat(y1, "y1")
+    T2, D2, s2 = _mat(y2, "y2")
+    if (T1, D1) != (T, D) or (T2, D2) != (T, D) or y1.dtype != y2.dtype:
+        raise ValueError("y1 and y2 must be [T, D] of one dtype")
+    for n, v in (("w1", w1), ("w2", w2), ("post_w", post_w), ("pre_w", pre_w)):
+        _f32(v, n, (D,))
+    h = torch.empty(T, D, dtype=y1.dtype, device=dev) if pre_w is not None else None
+    _lib.check(lib.b2_sandwich_norm_pair(_ptr(x), T, D, _ptr(y1), s1, _ptr(w1), _ptr(y2), s2, _ptr(w2), float(pair_scale), _ptr(post_w),
+                                         _ptr(pre_w), float(eps), _ptr(h), D, _act(y1, "y1"), _stream(dev)))
+    return h
+
+
 def row_norm(x: torch.Tensor, weight: Optional[torch.Tensor], eps: float) -> torch.Tensor:
     """x / sqrt(mean(x^2) + eps) * weight over activation rows [T, n] (a column slice of a wider row is fine; statistics in
     fp32).  Returns a contiguous [T, n] of x's dtype.  b2_row_norm."""
@@ -1335,15 +1403,27 @@ def softcap_(z: torch.Tensor, cap: float) -> torch.Tensor:
     return z
 
 
+def three_zone_frequencies(f: torch.Tensor, factor: float, low: float, high: float, original: float) -> torch.Tensor:
+    """Llama-3.1 frequency scaling of angles per position f (fp64): wavelengths below original / high stay, those above
+    original / low are slowed by `factor`, a blend linear in original / wavelength between the two."""
+    turns = original * f / (2.0 * math.pi)                      # original / wavelength
+    s = (turns - low) / (high - low)
+    mid = (1.0 - s) * f / factor + s * f
+    return torch.where(turns > high, f, torch.where(turns < low, f / factor, mid))
+
+
 def rotary_table(max_pos: int, dims: int, base: float, scaling: Optional[dict], device) -> torch.Tensor:
     """fp32 [max_pos, dims] = cos | sin halves per position (column i: pair i of either pair layout), angles in fp64.
     scaling {factor, original, fast, slow} (YaRN): pairs that complete more than `fast` turns within `original` positions
     keep their frequency, pairs below `slow` turns are slowed by `factor`, a linear ramp over the pair index between the
-    two; cos and sin carry the magnitude 0.1 ln(factor) + 1."""
+    two; cos and sin carry the magnitude 0.1 ln(factor) + 1.  scaling {factor, original, low, high}: three_zone_frequencies,
+    no magnitude."""
     half = dims // 2
     f = base ** (-2.0 * torch.arange(half, dtype=torch.float64) / dims)
     mag = 1.0
-    if scaling:
+    if scaling and "high" in scaling:
+        f = three_zone_frequencies(f, *(float(scaling[k]) for k in ("factor", "low", "high", "original")))
+    elif scaling:
         factor, original = float(scaling["factor"]), float(scaling["original"])
 
         def turn_dim(t):

@@ -10,9 +10,14 @@
 //     (window = 0: no window).  A query then reads the kept keys and its window's keys and nothing between them,
 //   * a sigmoid gate per (token, head) on the head's output,
 //   * the weight of a visible key: its share of the softmax, or (B2_WEIGHT_SIGMOID) sigmoid(score + head_bias[h]), a number
-//     of its own that no other key changes -- no maximum, no denominator, and a sink has no meaning.
+//     of its own that no other key changes -- no maximum, no denominator, and a sink has no meaning,
+//   * a cap on the scores: s <- cap * tanh(s / cap) before the mask and the softmax (cap = 0: none),
+//   * two maps per head (differential attention): a head holds two queries and two keys of size dk, each pair of them is a
+//     softmax attention of its own over the head's values, and the head's output is a1 - lambda * a2, divided by its own root
+//     mean square over dv (eps inside the root) and multiplied by a constant.  The two maps of a head are neighbours in q
+//     [T, H, maps, dk] and in the K pool; they are walked together, so a value row is read once for both.
 // Key size dk and value size dv are independent; K and V live in separate paged pools
-//   k_cache [num_blocks, G, bs, dk],  v_cache [num_blocks, G, bs, dv]      (activation type).
+//   k_cache [num_blocks, G * maps, bs, dk],  v_cache [num_blocks, G, bs, dv]      (activation type).
 //
 //   b2_qknorm_cache      per token: q heads normalised into q_out; k heads normalised and written to the K pool, v copied
 //                        to the V pool, through the token's slot (slot < 0 skips the write).
@@ -22,7 +27,8 @@
 //   b2_qk_rope_cache     rows [q | k] or [q | k | v]: the first rot_dims entries of every q and k head are rotated by the
 //                        token's position (pairs (i, i + rot_dims/2) or (2i, 2i + 1); fp32 table [max_pos, rot_dims] =
 //                        cos | sin halves), q to q_out, rotated k to the K pool; the V pool receives v, or, for designs
-//                        whose values ARE the keys, the k heads as projected (before the rotation).
+//                        whose values ARE the keys, the k heads as projected (before the rotation).  The value heads may be
+//                        fewer than the key heads (two key maps over one set of values).
 //   b2_qk_norm_rope_cache  rows [q | k | v]: all of q (H * dk numbers) and all of k (G * dk) are RMS-normed as one row each,
 //                        before the split into heads (fp32 weights of those sizes), then rotated and written as above; the
 //                        numbers stay in fp32 between the norm and the rotation.
@@ -88,7 +94,7 @@ __device__ __forceinline__ void qk_row_scales(const T* src, int nq, int nk, floa
 // Rows [q | k] (+ [v]): partial rotation of the q and k heads, K (rotated) and V pool writes; see the file comment.  NORM:
 // q and k are first normed over their whole rows.
 template <typename T, bool NORM>
-__global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, int G, int dk, int dv, bool v_from_k,
+__global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, int G, int Gv, int dk, int dv, bool v_from_k,
                                      int rot_dims, bool interleaved, const int32_t* __restrict__ positions,
                                      const float* __restrict__ cos_sin, int max_pos, const int64_t* __restrict__ slots, int bs,
                                      const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
@@ -127,9 +133,9 @@ __global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stri
     }
     if (slot < 0) return;
     const T* vsrc = v_from_k ? src + (size_t)H * dk : src + (size_t)(H + G) * dk;
-    for (int idx = threadIdx.x; idx < G * dv; idx += blockDim.x) {
+    for (int idx = threadIdx.x; idx < Gv * dv; idx += blockDim.x) {
         const int g = idx / dv, i = idx % dv;
-        v_cache[(((size_t)blk * G + g) * bs + off) * dv + i] = vsrc[idx];
+        v_cache[(((size_t)blk * Gv + g) * bs + off) * dv + i] = vsrc[idx];
     }
 }
 
@@ -137,7 +143,7 @@ __global__ void qk_rope_cache_kernel(const T* __restrict__ qkv, int64_t qkv_stri
 // eight in the (i, i + rot_dims/2) layout so that a group of four and its partners never straddle the halves.
 template <typename T, bool NORM>
 __global__ void __launch_bounds__(256)
-qk_rope_cache_vec_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, int G, int dk, int dv, bool v_from_k, int rot_dims,
+qk_rope_cache_vec_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, int G, int Gv, int dk, int dv, bool v_from_k, int rot_dims,
                          bool interleaved, const int32_t* __restrict__ positions, const float* __restrict__ cos_sin, int max_pos,
                          const int64_t* __restrict__ slots, int bs, const float* __restrict__ q_w, const float* __restrict__ k_w,
                          float eps, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache) {
@@ -193,11 +199,11 @@ qk_rope_cache_vec_kernel(const T* __restrict__ qkv, int64_t qkv_stride, int H, i
     if (slot < 0) return;
     const T* vsrc = v_from_k ? src + (size_t)H * dk : src + (size_t)(H + G) * dk;
     const int pv = dv / 4;
-    for (int idx = threadIdx.x; idx < G * pv; idx += blockDim.x) {
+    for (int idx = threadIdx.x; idx < Gv * pv; idx += blockDim.x) {
         const int g = idx / pv, i = (idx % pv) * 4;
         float x[4];
         b2::ld4(vsrc + (size_t)g * dv + i, x);
-        b2::st4(v_cache + (((size_t)blk * G + g) * bs + off) * dv + i, x);
+        b2::st4(v_cache + (((size_t)blk * Gv + g) * bs + off) * dv + i, x);
     }
 }
 
@@ -251,14 +257,26 @@ __global__ void qknorm_cache_kernel(const T* __restrict__ qkv, int64_t qkv_strid
 // sigmoid of a score that is already in the exponent of 2
 __device__ __forceinline__ float sigmoid2_f(float x2) { return __fdividef(1.f, 1.f + b2::fast_exp2(-x2)); }
 
-template <typename T, bool SIG>
+// What happens to a score before its weight is taken, and to a head's output after the values are summed.
+struct HeadShape {
+    float cap;               // > 0: scores become cap * tanh(score / cap)
+    float lambda;            // two maps: output = a1 - lambda * a2 ...
+    float eps, out_scale;    // ... / sqrt(mean(output^2) + eps) * out_scale
+};
+// cap * tanh(s / cap); tanh x = 1 - 2 / (1 + e^2x), whose absolute error (times cap) is that of one fp32 rounding
+__device__ __forceinline__ float cap_score(float s, float cap, float e_scale) {
+    return fmaf(-cap, __fdividef(2.f, 1.f + b2::fast_exp2(s * e_scale)), cap);
+}
+__device__ __forceinline__ float cap_score_exact(float s, float cap) { return cap * tanhf(s / cap); }
+
+template <typename T, bool SIG, int MAPS>
 __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                                        const int32_t* __restrict__ block_tables, int max_nb,
                                        const int32_t* __restrict__ cu_q, const int32_t* __restrict__ ctx_start, int n_seq,
                                        int rows, int H, int G, int dk, int dv, int bs, float scale, int chunk, int window,
                                        int keep_first, float sink, float sink_logit, const float* __restrict__ sink_logits,
                                        const float* __restrict__ head_bias, const T* __restrict__ gate, int64_t gate_stride,
-                                       int skip_rows_from, T* __restrict__ out, int64_t out_stride) {
+                                       HeadShape hs, int skip_rows_from, T* __restrict__ out, int64_t out_stride) {
     extern __shared__ float q_sm[];                  // [warps, dk]
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const int item = blockIdx.x * (blockDim.x >> 5) + wid;       // (row, head)
@@ -276,53 +294,72 @@ __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restr
     const KeySpan span = key_span(pos, pos, chunk, window, keep_first);
     const int g = hh / (H / G);
     float* qs = q_sm + (size_t)wid * dk;
-    const T* qv = q + (size_t)item * dk;
-    for (int i = lane; i < dk; i += 32) qs[i] = b2::ld(qv + i) * scale;
-    __syncwarp();
     const int32_t* bt = block_tables + (size_t)seq * max_nb;
-    float m = sink > 0.f ? (sink_logits ? sink_logits[hh] : sink_logit) : -INFINITY, l = sink;      // the sink seeds the running maximum and denominator
     const float bias = SIG && head_bias ? head_bias[hh] : 0.f;
+    float first[MAPS > 1 ? kMaxDvPerLane : 1];       // the first map's output
     float acc[kMaxDvPerLane];
+    float inv = 1.f;
 #pragma unroll
-    for (int c = 0; c < kMaxDvPerLane; ++c) acc[c] = 0.f;
-    for (int c0 = 0; c0 < span.n; c0 += 32) {
-        const bool in = c0 + lane < span.n;
-        const int j = span.key(c0 + lane);
-        float s = -INFINITY;
-        size_t vbase = 0;
-        if (in) {
-            const size_t tile = ((size_t)bt[j / bs] * G + g) * bs + (j % bs);
-            const T* kr = k_cache + tile * dk;
-            vbase = tile * dv;
-            float d = 0.f;
-            for (int i = 0; i < dk; ++i) d = fmaf(qs[i], b2::ld(kr + i), d);
-            s = d;
-        }
-        float p;
-        if (SIG) {
-            p = in ? b2::sigmoid_f(s + bias) : 0.f;
-        } else {
-            const float m_new = fmaxf(m, b2::warp_max(s));
-            const float corr = m == -INFINITY ? 0.f : __expf(m - m_new);
-            p = in ? __expf(s - m_new) : 0.f;
-            l = l * corr + b2::warp_sum(p);
-            m = m_new;
+    for (int mp = 0; mp < MAPS; ++mp) {
+        const T* qv = q + ((size_t)item * MAPS + mp) * dk;
+        __syncwarp();
+        for (int i = lane; i < dk; i += 32) qs[i] = b2::ld(qv + i) * scale;
+        __syncwarp();
+        float m = sink > 0.f ? (sink_logits ? sink_logits[hh] : sink_logit) : -INFINITY, l = sink;      // the sink seeds the running maximum and denominator
 #pragma unroll
-            for (int c = 0; c < kMaxDvPerLane; ++c) acc[c] *= corr;
-        }
-        const int nk = min(32, span.n - c0);
-        for (int kk = 0; kk < nk; ++kk) {
-            const float pk = __shfl_sync(0xffffffffu, p, kk);
-            const size_t vb = __shfl_sync(0xffffffffu, (unsigned long long)vbase, kk);
-            const T* vr = v_cache + vb;
+        for (int c = 0; c < kMaxDvPerLane; ++c) acc[c] = 0.f;
+        for (int c0 = 0; c0 < span.n; c0 += 32) {
+            const bool in = c0 + lane < span.n;
+            const int j = span.key(c0 + lane);
+            float s = -INFINITY;
+            size_t vbase = 0;
+            if (in) {
+                const size_t page = bt[j / bs];
+                const T* kr = k_cache + ((page * (G * MAPS) + g * MAPS + mp) * bs + (j % bs)) * dk;
+                vbase = ((page * G + g) * bs + (j % bs)) * dv;
+                float d = 0.f;
+                for (int i = 0; i < dk; ++i) d = fmaf(qs[i], b2::ld(kr + i), d);
+                s = hs.cap > 0.f ? cap_score_exact(d, hs.cap) : d;
+            }
+            float p;
+            if (SIG) {
+                p = in ? b2::sigmoid_f(s + bias) : 0.f;
+            } else {
+                const float m_new = fmaxf(m, b2::warp_max(s));
+                const float corr = m == -INFINITY ? 0.f : __expf(m - m_new);
+                p = in ? __expf(s - m_new) : 0.f;
+                l = l * corr + b2::warp_sum(p);
+                m = m_new;
 #pragma unroll
-            for (int c = 0; c < kMaxDvPerLane; ++c) {
-                const int i = lane + 32 * c;
-                if (i < dv) acc[c] = fmaf(pk, b2::ld(vr + i), acc[c]);
+                for (int c = 0; c < kMaxDvPerLane; ++c) acc[c] *= corr;
+            }
+            const int nk = min(32, span.n - c0);
+            for (int kk = 0; kk < nk; ++kk) {
+                const float pk = __shfl_sync(0xffffffffu, p, kk);
+                const size_t vb = __shfl_sync(0xffffffffu, (unsigned long long)vbase, kk);
+                const T* vr = v_cache + vb;
+#pragma unroll
+                for (int c = 0; c < kMaxDvPerLane; ++c) {
+                    const int i = lane + 32 * c;
+                    if (i < dv) acc[c] = fmaf(pk, b2::ld(vr + i), acc[c]);
+                }
             }
         }
+        inv = SIG ? 1.f : (l > 0.f ? 1.f / l : 0.f);
+        if (MAPS > 1 && mp == 0) {
+#pragma unroll
+            for (int c = 0; c < kMaxDvPerLane; ++c) first[MAPS > 1 ? c : 0] = acc[c] * inv;
+        }
     }
-    float inv = SIG ? 1.f : (l > 0.f ? 1.f / l : 0.f);
+    if (MAPS > 1) {
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < kMaxDvPerLane; ++c) {
+            acc[c] = first[MAPS > 1 ? c : 0] - hs.lambda * (acc[c] * inv);
+            ss = fmaf(acc[c], acc[c], ss);           // columns past dv hold zeros
+        }
+        inv = rsqrtf(b2::warp_sum(ss) / (float)dv + hs.eps) * hs.out_scale;
+    }
     if (gate) inv *= b2::sigmoid_f(b2::ld(gate + (size_t)row * gate_stride + hh));
 #pragma unroll
     for (int c = 0; c < kMaxDvPerLane; ++c) {
@@ -336,29 +373,31 @@ __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restr
 // query heads of that kv head, so K and V are read once per group instead of once per head.  Four warps share the visible
 // keys 32 at a time (a lane per key, 16-byte loads of its K row, one dot product per query head), keep an online softmax
 // per head, accumulate P.V with a lane per pair of value columns, and merge through shared memory; the sink enters
-// through warp 0's initial state.  Up to kGroupMaxHeads query heads per pass (more: further passes over the keys).
+// through warp 0's initial state.  Up to kGroupMaxHeads query heads per pass (more: further passes over the keys).  With two
+// maps the pass holds the heads' maps one after the other (an even number) and a key's two halves lie side by side in the tile.
 constexpr int kGroupMaxHeads = 8, kGroupMaxPairs = 4;      // dv <= 256
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(b2::smem_u32(dst)), "l"(src) : "memory");
 }
 
-template <bool SIG>
+template <bool SIG, int MAPS>
 __global__ void __launch_bounds__(128)
 chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                              const __nv_bfloat16* __restrict__ v_cache, const int32_t* __restrict__ block_tables, int max_nb,
                              const int32_t* __restrict__ cu_q, const int32_t* __restrict__ ctx_start, int n_seq, int H, int G,
                              int dk, int dv, int bs, float scale, int chunk, int window, int keep_first, float sink,
                              float sink_logit, const float* __restrict__ sink_logits, const float* __restrict__ head_bias,
-                             const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, int skip_rows_from,
+                             const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, HeadShape hs, int skip_rows_from,
                              __nv_bfloat16* __restrict__ out, int64_t out_stride) {
-    // q [QH][dk] | per warp: m [QH], l [QH], acc [QH][dv] | per warp: K tile [32][dk + 8], V tile [32][dv] (bf16)
+    // q [QH][dk] | per warp: m [QH], l [QH], acc [QH][dv] | per warp: K tile [32][MAPS * dk + 8], V tile [32][dv] (bf16)
     extern __shared__ __align__(16) float grp_sm[];
     const int row = blockIdx.x, g = blockIdx.y;
     const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
     const int seq = b2::seq_of_row(cu_q, n_seq, row);
     const int ctx = ctx_start[seq];
-    const int QHall = H / G;
+    const int QHall = H / G;                               // query heads of this key head
+    const int VHall = QHall * MAPS;                        // ... each with its maps
     if (skip_rows_from > 0 && ctx >= 0 && cu_q[seq + 1] - cu_q[seq] >= skip_rows_from) return;    // the tile kernel's
     if (ctx < 0) {
         for (int i = tid; i < QHall * dv; i += 128)
@@ -369,23 +408,23 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
     const KeySpan span = key_span(pos, pos, chunk, window, keep_first);
     const int32_t* bt = block_tables + (size_t)seq * max_nb;
     const int npairs = dv / 2;
-    for (int h0 = 0; h0 < QHall; h0 += kGroupMaxHeads) {
-        const int QH = min(kGroupMaxHeads, QHall - h0);
+    for (int h0 = 0; h0 < VHall; h0 += kGroupMaxHeads) {
+        const int QH = min(kGroupMaxHeads, VHall - h0);
         float* qs = grp_sm;
         float* part = grp_sm + kGroupMaxHeads * dk;
-        const int ldk = dk + 8;                            // 16 bytes of padding: the lanes' rows spread over the banks
+        const int ldk = MAPS * dk + 8;                     // 16 bytes of padding: the lanes' rows spread over the banks
         __nv_bfloat16* kt = reinterpret_cast<__nv_bfloat16*>(part + 4 * kGroupMaxHeads * (2 + dv)) + (size_t)w * 32 * (ldk + dv);
         __nv_bfloat16* vt = kt + 32 * ldk;
         __syncthreads();                                   // a previous pass is done with the shared memory
         for (int i = tid; i < QH * dk; i += 128)
-            qs[i] = __bfloat162float(q[((size_t)row * H + (size_t)g * QHall + h0) * dk + i]) * scale;
+            qs[i] = __bfloat162float(q[((size_t)row * H * MAPS + (size_t)g * VHall + h0) * dk + i]) * scale;
         __syncthreads();
         float m[kGroupMaxHeads], l[kGroupMaxHeads], acc[kGroupMaxHeads][kGroupMaxPairs][2];
 #pragma unroll
         for (int h = 0; h < kGroupMaxHeads; ++h) {
-            m[h] = (w == 0 && sink > 0.f) ? (sink_logits ? sink_logits[g * QHall + h0 + min(h, QH - 1)] : sink_logit) : -INFINITY;
+            m[h] = (w == 0 && sink > 0.f) ? (sink_logits ? sink_logits[g * QHall + (h0 + min(h, QH - 1)) / MAPS] : sink_logit) : -INFINITY;
             l[h] = w == 0 ? sink : 0.f;
-            if (SIG) m[h] = head_bias ? head_bias[g * QHall + h0 + min(h, QH - 1)] : 0.f;      // holds the head's bias instead
+            if (SIG) m[h] = head_bias ? head_bias[g * QHall + (h0 + min(h, QH - 1)) / MAPS] : 0.f;      // holds the head's bias instead
 #pragma unroll
             for (int c = 0; c < kGroupMaxPairs; ++c) acc[h][c][0] = acc[h][c][1] = 0.f;
         }
@@ -397,9 +436,10 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
             // the warp's 32 keys: K and V rows gathered from the pages with every 16-byte copy in flight at once
             const int nk = min(32, span.n - c0);
             __syncwarp();                                  // the previous tile has been read
-            for (int idx = lane; idx < nk * (dk / 8); idx += 32) {
-                const int key = idx / (dk / 8), c = (idx % (dk / 8)) * 8, jk = span.key(c0 + key);
-                cp_async16(kt + key * ldk + c, k_cache + (((size_t)bt[jk / bs] * G + g) * bs + jk % bs) * dk + c);
+            for (int idx = lane; idx < nk * MAPS * (dk / 8); idx += 32) {
+                const int part_ = idx / (dk / 8), c = (idx % (dk / 8)) * 8, key = part_ / MAPS, mp = part_ % MAPS, jk = span.key(c0 + key);
+                cp_async16(kt + key * ldk + mp * dk + c,
+                           k_cache + (((size_t)bt[jk / bs] * (G * MAPS) + g * MAPS + mp) * bs + jk % bs) * dk + c);
             }
             for (int idx = lane; idx < nk * (dv / 8); idx += 32) {
                 const int key = idx / (dv / 8), c = (idx % (dv / 8)) * 8, jk = span.key(c0 + key);
@@ -409,27 +449,35 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
             asm volatile("cp.async.wait_group 0;" ::: "memory");
             __syncwarp();
             if (valid) {
-                const __nv_bfloat16* kr = kt + lane * ldk;
-                for (int c = 0; c < dk; c += 8) {
-                    const uint4 raw = *reinterpret_cast<const uint4*>(kr + c);
-                    const uint32_t wds[4] = {raw.x, raw.y, raw.z, raw.w};
-                    float kf[8];
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        kf[2 * e] = __uint_as_float(wds[e] << 16);
-                        kf[2 * e + 1] = __uint_as_float(wds[e] & 0xffff0000u);
-                    }
+                for (int mp = 0; mp < MAPS; ++mp) {
+                    const __nv_bfloat16* kr = kt + lane * ldk + mp * dk;
+                    for (int c = 0; c < dk; c += 8) {
+                        const uint4 raw = *reinterpret_cast<const uint4*>(kr + c);
+                        const uint32_t wds[4] = {raw.x, raw.y, raw.z, raw.w};
+                        float kf[8];
 #pragma unroll
-                    for (int h = 0; h < kGroupMaxHeads; ++h) {
-                        if (h < QH) {
-                            const float4 qa = *reinterpret_cast<const float4*>(qs + h * dk + c);
-                            const float4 qb = *reinterpret_cast<const float4*>(qs + h * dk + c + 4);
-                            sc[h] = fmaf(qa.x, kf[0], sc[h]); sc[h] = fmaf(qa.y, kf[1], sc[h]);
-                            sc[h] = fmaf(qa.z, kf[2], sc[h]); sc[h] = fmaf(qa.w, kf[3], sc[h]);
-                            sc[h] = fmaf(qb.x, kf[4], sc[h]); sc[h] = fmaf(qb.y, kf[5], sc[h]);
-                            sc[h] = fmaf(qb.z, kf[6], sc[h]); sc[h] = fmaf(qb.w, kf[7], sc[h]);
+                        for (int e = 0; e < 4; ++e) {
+                            kf[2 * e] = __uint_as_float(wds[e] << 16);
+                            kf[2 * e + 1] = __uint_as_float(wds[e] & 0xffff0000u);
+                        }
+#pragma unroll
+                        for (int h = mp; h < kGroupMaxHeads; h += MAPS) {
+                            if (h < QH) {
+                                const float4 qa = *reinterpret_cast<const float4*>(qs + h * dk + c);
+                                const float4 qb = *reinterpret_cast<const float4*>(qs + h * dk + c + 4);
+                                sc[h] = fmaf(qa.x, kf[0], sc[h]); sc[h] = fmaf(qa.y, kf[1], sc[h]);
+                                sc[h] = fmaf(qa.z, kf[2], sc[h]); sc[h] = fmaf(qa.w, kf[3], sc[h]);
+                                sc[h] = fmaf(qb.x, kf[4], sc[h]); sc[h] = fmaf(qb.y, kf[5], sc[h]);
+                                sc[h] = fmaf(qb.z, kf[6], sc[h]); sc[h] = fmaf(qb.w, kf[7], sc[h]);
+                            }
                         }
                     }
+                }
+                if (hs.cap > 0.f) {
+                    const float e_scale = 2.8853900817779268f / hs.cap;         // 2 log2(e) / cap
+#pragma unroll
+                    for (int h = 0; h < kGroupMaxHeads; ++h) sc[h] = cap_score(sc[h], hs.cap, e_scale);
                 }
             }
             float pr[kGroupMaxHeads];
@@ -497,8 +545,8 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
             }
         }
         __syncthreads();
-        for (int i = tid; i < QH * dv; i += 128) {
-            const int h = i / dv, col = i % dv;
+        // output of (virtual) head h at column col
+        auto merged = [&](int h, int col) {
             float M = -INFINITY, L = 0.f, O = 0.f;
             if (SIG) {
                 L = 1.f;
@@ -514,9 +562,33 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
                     O = fmaf(px[2 + col], f, O);
                 }
             }
-            float res = L > 0.f ? O / L : 0.f;
-            if (gate) res *= b2::sigmoid_f(__bfloat162float(gate[(size_t)row * gate_stride + (size_t)g * QHall + h0 + h]));
-            out[(size_t)row * out_stride + ((size_t)g * QHall + h0 + h) * dv + col] = __float2bfloat16_rn(res);
+            return L > 0.f ? O / L : 0.f;
+        };
+        if (MAPS == 1) {
+            for (int i = tid; i < QH * dv; i += 128) {
+                const int h = i / dv, col = i % dv;
+                float res = merged(h, col);
+                if (gate) res *= b2::sigmoid_f(__bfloat162float(gate[(size_t)row * gate_stride + (size_t)g * QHall + h0 + h]));
+                out[(size_t)row * out_stride + ((size_t)g * QHall + h0 + h) * dv + col] = __float2bfloat16_rn(res);
+            }
+        } else {
+            for (int h = w; h < QH / MAPS; h += 4) {           // a warp per head: the norm runs over its dv columns
+                const size_t head = (size_t)g * QHall + h0 / MAPS + h;
+                float v[2 * kGroupMaxPairs], ss = 0.f;
+#pragma unroll
+                for (int c = 0; c < 2 * kGroupMaxPairs; ++c) {
+                    const int col = lane + 32 * c;
+                    v[c] = col < dv ? merged(h * MAPS, col) - hs.lambda * merged(h * MAPS + MAPS - 1, col) : 0.f;
+                    ss = fmaf(v[c], v[c], ss);
+                }
+                float inv = rsqrtf(b2::warp_sum(ss) / (float)dv + hs.eps) * hs.out_scale;
+                if (gate) inv *= b2::sigmoid_f(__bfloat162float(gate[(size_t)row * gate_stride + head]));
+#pragma unroll
+                for (int c = 0; c < 2 * kGroupMaxPairs; ++c) {
+                    const int col = lane + 32 * c;
+                    if (col < dv) out[(size_t)row * out_stride + head * dv + col] = __float2bfloat16_rn(v[c] * inv);
+                }
+            }
         }
     }
 }
@@ -532,16 +604,16 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
 // kernel above.
 constexpr int kTQ = 64, kTK = 64, kTileMinRows = 16;
 
-template <int DKT, int DVT, bool SIG>
+template <int DKT, int DVT, bool SIG, int MAPS>
 __global__ void __launch_bounds__(128)
 chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                             const __nv_bfloat16* __restrict__ v_cache, const int32_t* __restrict__ block_tables, int max_nb,
                             const int32_t* __restrict__ cu_q, const int32_t* __restrict__ ctx_start, int n_seq, int H, int G,
                             int bs, float scale_log2, int chunk, int window, int keep_first, float sink,
                             float sink_logit_log2, const float* __restrict__ sink_logits, const float* __restrict__ head_bias,
-                            const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, __nv_bfloat16* __restrict__ out,
+                            const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, HeadShape hs, __nv_bfloat16* __restrict__ out,
                             int64_t out_stride) {
-    constexpr int DK = 16 * DKT, DV = 16 * DVT, LDK = DK + 8, LDV = DV + 8;
+    constexpr int DK = 16 * DKT, DV = 16 * DVT, LDK = MAPS * DK + 8, LDV = DV + 8;
     extern __shared__ __align__(16) unsigned char tile_smem[];
     __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(tile_smem);      // [64][LDK]
     __nv_bfloat16* k_sm = q_sm + kTQ * LDK;                                 // [2][64][LDK]
@@ -571,10 +643,10 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     const KeySpan span = key_span(p0, p_last, chunk, window, keep_first);
     const int32_t* bt = block_tables + (size_t)seq * max_nb;
 
-    for (int idx = tid; idx < kTQ * (DK / 8); idx += 128) {
-        const int r = idx / (DK / 8), c = (idx % (DK / 8)) * 8;
+    for (int idx = tid; idx < kTQ * (MAPS * DK / 8); idx += 128) {
+        const int r = idx / (MAPS * DK / 8), c = (idx % (MAPS * DK / 8)) * 8;
         uint4 v = make_uint4(0, 0, 0, 0);
-        if (r < rows) v = *reinterpret_cast<const uint4*>(q + ((size_t)(r0 + r) * H + hh) * DK + c);
+        if (r < rows) v = *reinterpret_cast<const uint4*>(q + ((size_t)(r0 + r) * H + hh) * (MAPS * DK) + c);
         *reinterpret_cast<uint4*>(q_sm + r * LDK + c) = v;
     }
     const int gq = lane >> 2, tq = lane & 3;
@@ -584,12 +656,17 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     const int w_clo = chunk > 0 ? (w_first / chunk) * chunk : 0;
     const int w_lo = window > 0 ? max(w_clo, w_first - window + 1) : w_clo;   // the lowest key of the warp's rows' windows
     if (sink_logits) sink_logit_log2 = sink_logits[hh] * 1.4426950408889634f;
-    float m0 = sink > 0.f ? sink_logit_log2 : -INFINITY, m1 = m0;
-    float l0 = tq == 0 ? sink : 0.f, l1 = l0;                               // partial sums per lane; the sink counted once
-    const float bias_log2 = SIG && head_bias ? head_bias[hh] * 1.4426950408889634f : 0.f;
-    float o[2 * DVT][4];
+    float m0[MAPS], m1[MAPS], l0[MAPS], l1[MAPS];                           // partial sums per lane; the sink counted once
+    float o[MAPS][2 * DVT][4];
 #pragma unroll
-    for (int n = 0; n < 2 * DVT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    for (int mp = 0; mp < MAPS; ++mp) {
+        m0[mp] = m1[mp] = sink > 0.f ? sink_logit_log2 : -INFINITY;
+        l0[mp] = l1[mp] = tq == 0 ? sink : 0.f;
+#pragma unroll
+        for (int n = 0; n < 2 * DVT; ++n) o[mp][n][0] = o[mp][n][1] = o[mp][n][2] = o[mp][n][3] = 0.f;
+    }
+    const float bias_log2 = SIG && head_bias ? head_bias[hh] * 1.4426950408889634f : 0.f;
+    const float cap_log2 = hs.cap * 1.4426950408889634f, cap_e = hs.cap > 0.f ? 2.f / hs.cap : 0.f;
     const uint32_t q_base = b2::smem_u32(q_sm), k_base0 = b2::smem_u32(k_sm), v_base0 = b2::smem_u32(v_sm);
 
     const int ld_key = tid >> 1, ld_half = tid & 1;
@@ -599,16 +676,19 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         __nv_bfloat16* vd = v_sm + (buf * kTK + ld_key) * LDV;
         if (j <= p_last) {
             const int page = j / bs;
-            const size_t row = ((size_t)bt[page] * G + g) * bs + (j - page * bs);
-            const __nv_bfloat16* ks = k_cache + row * DK;
-            const __nv_bfloat16* vs = v_cache + row * DV;
+            const size_t blk = bt[page], off = j - page * bs;
+            const __nv_bfloat16* vs = v_cache + ((blk * G + g) * bs + off) * DV;
 #pragma unroll
-            for (int c = 0; c < DKT; ++c) cp_async16(kd + (2 * c + ld_half) * 8, ks + (2 * c + ld_half) * 8);
+            for (int mp = 0; mp < MAPS; ++mp) {
+                const __nv_bfloat16* ks = k_cache + ((blk * (G * MAPS) + g * MAPS + mp) * bs + off) * DK;
+#pragma unroll
+                for (int c = 0; c < DKT; ++c) cp_async16(kd + mp * DK + (2 * c + ld_half) * 8, ks + (2 * c + ld_half) * 8);
+            }
 #pragma unroll
             for (int c = 0; c < DVT; ++c) cp_async16(vd + (2 * c + ld_half) * 8, vs + (2 * c + ld_half) * 8);
         } else {
 #pragma unroll
-            for (int c = 0; c < DKT; ++c) *reinterpret_cast<uint4*>(kd + (2 * c + ld_half) * 8) = make_uint4(0, 0, 0, 0);
+            for (int c = 0; c < MAPS * DKT; ++c) *reinterpret_cast<uint4*>(kd + (2 * c + ld_half) * 8) = make_uint4(0, 0, 0, 0);
 #pragma unroll
             for (int c = 0; c < DVT; ++c) *reinterpret_cast<uint4*>(vd + (2 * c + ld_half) * 8) = make_uint4(0, 0, 0, 0);
         }
@@ -631,114 +711,159 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         const bool full = kv0 + kTK <= span.n && j_max <= w_first && (chunk <= 0 || j_min >= (w_last / chunk) * chunk) &&
                           (window <= 0 || w_last - j_min < window || j_max < keep_first);
         if (!none) {
-            float sc[8][4];
 #pragma unroll
-            for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+            for (int mp = 0; mp < MAPS; ++mp) {
+                float sc[8][4];
 #pragma unroll
-            for (int kk = 0; kk < DKT; ++kk) {
-                uint32_t a0, a1, a2, a3;
-                b2::ldmatrix_x4(q_base + 2u * ((w * 16 + (lane & 15)) * LDK + kk * 16 + (lane >> 4) * 8), a0, a1, a2, a3);
+                for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
 #pragma unroll
-                for (int n2 = 0; n2 < 4; ++n2) {
-                    uint32_t b0, b1, b2_, b3;
-                    const int key = n2 * 16 + (lane >> 4) * 8 + (lane & 7), dim = kk * 16 + ((lane >> 3) & 1) * 8;
-                    b2::ldmatrix_x4(k_base + 2u * (key * LDK + dim), b0, b1, b2_, b3);
-                    b2::mma_bf16_16816(sc[2 * n2], a0, a1, a2, a3, b0, b1);
-                    b2::mma_bf16_16816(sc[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
+                for (int kk = 0; kk < DKT; ++kk) {
+                    uint32_t a0, a1, a2, a3;
+                    b2::ldmatrix_x4(q_base + 2u * ((w * 16 + (lane & 15)) * LDK + mp * DK + kk * 16 + (lane >> 4) * 8), a0, a1, a2, a3);
+#pragma unroll
+                    for (int n2 = 0; n2 < 4; ++n2) {
+                        uint32_t b0, b1, b2_, b3;
+                        const int key = n2 * 16 + (lane >> 4) * 8 + (lane & 7), dim = mp * DK + kk * 16 + ((lane >> 3) & 1) * 8;
+                        b2::ldmatrix_x4(k_base + 2u * (key * LDK + dim), b0, b1, b2_, b3);
+                        b2::mma_bf16_16816(sc[2 * n2], a0, a1, a2, a3, b0, b1);
+                        b2::mma_bf16_16816(sc[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
+                    }
                 }
-            }
-            if (SIG) {                                                          // every weight by itself: nothing to rescale
-#pragma unroll
-                for (int n = 0; n < 8; ++n) {
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) sc[n][e] = sigmoid2_f(fmaf(sc[n][e], scale_log2, bias_log2));
-                }
-                if (!full) {
+                if (SIG) {                                                          // every weight by itself: nothing to rescale
 #pragma unroll
                     for (int n = 0; n < 8; ++n) {
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
-                            const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
-                            if (!ok) sc[n][e] = 0.f;
+                        for (int e = 0; e < 4; ++e) sc[n][e] = sigmoid2_f(fmaf(sc[n][e], scale_log2, bias_log2));
+                    }
+                    if (!full) {
+#pragma unroll
+                        for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
+                                const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
+                                if (!ok) sc[n][e] = 0.f;
+                            }
                         }
                     }
-                }
-            } else {
-                float mx0 = -INFINITY, mx1 = -INFINITY;
-#pragma unroll
-                for (int n = 0; n < 8; ++n) {
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) sc[n][e] *= scale_log2;
-                }
-                if (!full) {
+                } else {
+                    float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
                     for (int n = 0; n < 8; ++n) {
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
-                            const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
-                            if (!ok) sc[n][e] = -INFINITY;
+                        for (int e = 0; e < 4; ++e) sc[n][e] *= scale_log2;
+                    }
+                    if (hs.cap > 0.f) {
+#pragma unroll
+                        for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) sc[n][e] = cap_score(sc[n][e], cap_log2, cap_e);
                         }
+                    }
+                    if (!full) {
+#pragma unroll
+                        for (int n = 0; n < 8; ++n) {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const int j = span.key(kv0 + n * 8 + 2 * tq + (e & 1));
+                                const bool ok = e < 2 ? key_visible(i0, j, lo0, window, keep_first) : key_visible(i1, j, lo1, window, keep_first);
+                                if (!ok) sc[n][e] = -INFINITY;
+                            }
+                        }
+                    }
+#pragma unroll
+                    for (int n = 0; n < 8; ++n) {
+                        mx0 = fmaxf(mx0, fmaxf(sc[n][0], sc[n][1]));
+                        mx1 = fmaxf(mx1, fmaxf(sc[n][2], sc[n][3]));
+                    }
+                    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+                    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+                    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+                    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+                    const float mn0 = fmaxf(m0[mp], mx0), mn1 = fmaxf(m1[mp], mx1);
+                    const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
+                    const float c0 = b2::fast_exp2(m0[mp] - mu0), c1 = b2::fast_exp2(m1[mp] - mu1);             // exp2(-inf) = 0: nothing accumulated yet
+                    m0[mp] = mn0;
+                    m1[mp] = mn1;
+                    float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+                    for (int n = 0; n < 8; ++n) {
+                        sc[n][0] = b2::fast_exp2(sc[n][0] - mu0);
+                        sc[n][1] = b2::fast_exp2(sc[n][1] - mu0);
+                        sc[n][2] = b2::fast_exp2(sc[n][2] - mu1);
+                        sc[n][3] = b2::fast_exp2(sc[n][3] - mu1);
+                        s0 += sc[n][0] + sc[n][1];
+                        s1 += sc[n][2] + sc[n][3];
+                    }
+                    l0[mp] = l0[mp] * c0 + s0;
+                    l1[mp] = l1[mp] * c1 + s1;
+#pragma unroll
+                    for (int n = 0; n < 2 * DVT; ++n) {
+                        o[mp][n][0] *= c0;
+                        o[mp][n][1] *= c0;
+                        o[mp][n][2] *= c1;
+                        o[mp][n][3] *= c1;
                     }
                 }
 #pragma unroll
-                for (int n = 0; n < 8; ++n) {
-                    mx0 = fmaxf(mx0, fmaxf(sc[n][0], sc[n][1]));
-                    mx1 = fmaxf(mx1, fmaxf(sc[n][2], sc[n][3]));
-                }
-                mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-                mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-                mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-                mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-                const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-                const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
-                const float c0 = b2::fast_exp2(m0 - mu0), c1 = b2::fast_exp2(m1 - mu1);             // exp2(-inf) = 0: nothing accumulated yet
-                m0 = mn0;
-                m1 = mn1;
-                float s0 = 0.f, s1 = 0.f;
+                for (int ks = 0; ks < 4; ++ks) {
+                    const uint32_t a0 = b2::pack_bf16x2(sc[2 * ks][0], sc[2 * ks][1]), a1 = b2::pack_bf16x2(sc[2 * ks][2], sc[2 * ks][3]);
+                    const uint32_t a2 = b2::pack_bf16x2(sc[2 * ks + 1][0], sc[2 * ks + 1][1]),
+                                   a3 = b2::pack_bf16x2(sc[2 * ks + 1][2], sc[2 * ks + 1][3]);
 #pragma unroll
-                for (int n = 0; n < 8; ++n) {
-                    sc[n][0] = b2::fast_exp2(sc[n][0] - mu0);
-                    sc[n][1] = b2::fast_exp2(sc[n][1] - mu0);
-                    sc[n][2] = b2::fast_exp2(sc[n][2] - mu1);
-                    sc[n][3] = b2::fast_exp2(sc[n][3] - mu1);
-                    s0 += sc[n][0] + sc[n][1];
-                    s1 += sc[n][2] + sc[n][3];
-                }
-                l0 = l0 * c0 + s0;
-                l1 = l1 * c1 + s1;
-#pragma unroll
-                for (int n = 0; n < 2 * DVT; ++n) {
-                    o[n][0] *= c0;
-                    o[n][1] *= c0;
-                    o[n][2] *= c1;
-                    o[n][3] *= c1;
-                }
-            }
-#pragma unroll
-            for (int ks = 0; ks < 4; ++ks) {
-                const uint32_t a0 = b2::pack_bf16x2(sc[2 * ks][0], sc[2 * ks][1]), a1 = b2::pack_bf16x2(sc[2 * ks][2], sc[2 * ks][3]);
-                const uint32_t a2 = b2::pack_bf16x2(sc[2 * ks + 1][0], sc[2 * ks + 1][1]),
-                               a3 = b2::pack_bf16x2(sc[2 * ks + 1][2], sc[2 * ks + 1][3]);
-#pragma unroll
-                for (int n2 = 0; n2 < DVT; ++n2) {
-                    uint32_t b0, b1, b2_, b3;
-                    const int key = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), col = n2 * 16 + (lane >> 4) * 8;
-                    b2::ldmatrix_x4_trans(v_base + 2u * (key * LDV + col), b0, b1, b2_, b3);
-                    b2::mma_bf16_16816(o[2 * n2], a0, a1, a2, a3, b0, b1);
-                    b2::mma_bf16_16816(o[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
+                    for (int n2 = 0; n2 < DVT; ++n2) {
+                        uint32_t b0, b1, b2_, b3;
+                        const int key = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), col = n2 * 16 + (lane >> 4) * 8;
+                        b2::ldmatrix_x4_trans(v_base + 2u * (key * LDV + col), b0, b1, b2_, b3);
+                        b2::mma_bf16_16816(o[mp][2 * n2], a0, a1, a2, a3, b0, b1);
+                        b2::mma_bf16_16816(o[mp][2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
+                    }
                 }
             }
         }
         __syncthreads();                                                    // the tile is consumed: its buffer may be refilled
     }
-    l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
-    l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
-    l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
-    l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-    float inv0 = SIG ? 1.f : (l0 > 0.f ? 1.f / l0 : 0.f), inv1 = SIG ? 1.f : (l1 > 0.f ? 1.f / l1 : 0.f);
+    float inv0 = 1.f, inv1 = 1.f;
+#pragma unroll
+    for (int mp = 0; mp < MAPS; ++mp) {
+#pragma unroll
+        for (int x = 1; x < 4; x <<= 1) {
+            l0[mp] += __shfl_xor_sync(0xffffffffu, l0[mp], x);
+            l1[mp] += __shfl_xor_sync(0xffffffffu, l1[mp], x);
+        }
+        inv0 = SIG ? 1.f : (l0[mp] > 0.f ? 1.f / l0[mp] : 0.f);
+        inv1 = SIG ? 1.f : (l1[mp] > 0.f ? 1.f / l1[mp] : 0.f);
+        if (MAPS > 1) {
+            const float f0 = mp == 0 ? inv0 : -hs.lambda * inv0, f1 = mp == 0 ? inv1 : -hs.lambda * inv1;
+#pragma unroll
+            for (int n = 0; n < 2 * DVT; ++n) {
+                o[mp][n][0] *= f0;
+                o[mp][n][1] *= f0;
+                o[mp][n][2] *= f1;
+                o[mp][n][3] *= f1;
+            }
+        }
+    }
     const int ra = w * 16 + gq, rb = ra + 8;
+    if (MAPS > 1) {                                                         // the difference and its norm over the head's columns
+        float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+        for (int n = 0; n < 2 * DVT; ++n) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                o[0][n][e] += o[MAPS - 1][n][e];
+                if (e < 2) s0 = fmaf(o[0][n][e], o[0][n][e], s0);
+                else s1 = fmaf(o[0][n][e], o[0][n][e], s1);
+            }
+        }
+#pragma unroll
+        for (int x = 1; x < 4; x <<= 1) {
+            s0 += __shfl_xor_sync(0xffffffffu, s0, x);
+            s1 += __shfl_xor_sync(0xffffffffu, s1, x);
+        }
+        inv0 = rsqrtf(s0 / (float)DV + hs.eps) * hs.out_scale;
+        inv1 = rsqrtf(s1 / (float)DV + hs.eps) * hs.out_scale;
+    }
     if (gate) {
         if (ra < rows) inv0 *= b2::sigmoid_f(__bfloat162float(gate[(size_t)(r0 + ra) * gate_stride + hh]));
         if (rb < rows) inv1 *= b2::sigmoid_f(__bfloat162float(gate[(size_t)(r0 + rb) * gate_stride + hh]));
@@ -747,27 +872,27 @@ chunk_attention_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     for (int n = 0; n < 2 * DVT; ++n) {
         const int col = n * 8 + 2 * tq;
         if (ra < rows)
-            *reinterpret_cast<uint32_t*>(out + (size_t)(r0 + ra) * out_stride + hh * DV + col) = b2::pack_bf16x2(o[n][0] * inv0, o[n][1] * inv0);
+            *reinterpret_cast<uint32_t*>(out + (size_t)(r0 + ra) * out_stride + hh * DV + col) = b2::pack_bf16x2(o[0][n][0] * inv0, o[0][n][1] * inv0);
         if (rb < rows)
-            *reinterpret_cast<uint32_t*>(out + (size_t)(r0 + rb) * out_stride + hh * DV + col) = b2::pack_bf16x2(o[n][2] * inv1, o[n][3] * inv1);
+            *reinterpret_cast<uint32_t*>(out + (size_t)(r0 + rb) * out_stride + hh * DV + col) = b2::pack_bf16x2(o[0][n][2] * inv1, o[0][n][3] * inv1);
     }
 }
 
-template <int DKT, int DVT, bool SIG>
+template <int DKT, int DVT, bool SIG, int MAPS>
 int launch_tile(const void* q, const void* k_cache, const void* v_cache, const int32_t* block_tables, int max_nb,
                 const int32_t* cu_q, const int32_t* ctx_start, int n_seq, int T, int H, int G, int bs, float scale, int chunk,
                 int window, int keep_first, float sink, float sink_logit, const float* sink_logits, const float* head_bias,
-                const void* gate, int64_t gate_stride, void* out, int64_t out_stride, cudaStream_t st) {
+                const void* gate, int64_t gate_stride, const HeadShape& hs, void* out, int64_t out_stride, cudaStream_t st) {
     constexpr int DK = 16 * DKT, DV = 16 * DVT;
-    const size_t smem = (size_t)(kTQ * (DK + 8) + 2 * kTK * (DK + 8) + 2 * kTK * (DV + 8)) * sizeof(__nv_bfloat16);
-    auto kern = chunk_attention_tile_kernel<DKT, DVT, SIG>;
+    const size_t smem = (size_t)(kTQ * (MAPS * DK + 8) + 2 * kTK * (MAPS * DK + 8) + 2 * kTK * (DV + 8)) * sizeof(__nv_bfloat16);
+    auto kern = chunk_attention_tile_kernel<DKT, DVT, SIG, MAPS>;
     if (smem > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const int tiles = (T + kTQ - 1) / kTQ + n_seq;          // upper bound on sum(ceil(len / 64)); spare CTAs leave at once
     kern<<<dim3(tiles, H), 128, smem, st>>>(static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
                                            static_cast<const __nv_bfloat16*>(v_cache), block_tables, max_nb, cu_q, ctx_start,
                                            n_seq, H, G, bs, scale * 1.4426950408889634f, chunk, window, keep_first, sink,
                                            sink_logit * 1.4426950408889634f, sink_logits, head_bias,
-                                           static_cast<const __nv_bfloat16*>(gate), gate_stride, static_cast<__nv_bfloat16*>(out),
+                                           static_cast<const __nv_bfloat16*>(gate), gate_stride, hs, static_cast<__nv_bfloat16*>(out),
                                            out_stride);
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
@@ -812,18 +937,19 @@ extern "C" int b2_qk_rope_cache(const void* qkv, int64_t qkv_stride, int act_dty
                                 int v_from_k, int rot_dims, int interleaved, const int32_t* positions, const float* cos_sin,
                                 int max_pos, const int64_t* slots, int bs, void* q_out, void* k_cache, void* v_cache,
                                 void* stream) {
-    return b2_qk_norm_rope_cache(qkv, qkv_stride, act_dtype, T, H, G, dk, dv, v_from_k, nullptr, nullptr, 0.f, rot_dims, interleaved,
+    return b2_qk_norm_rope_cache(qkv, qkv_stride, act_dtype, T, H, G, G, dk, dv, v_from_k, nullptr, nullptr, 0.f, rot_dims, interleaved,
                                  positions, cos_sin, max_pos, slots, bs, q_out, k_cache, v_cache, stream);
 }
 
-extern "C" int b2_qk_norm_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, int T, int H, int G, int dk, int dv,
+extern "C" int b2_qk_norm_rope_cache(const void* qkv, int64_t qkv_stride, int act_dtype, int T, int H, int G, int Gv, int dk, int dv,
                                      int v_from_k, const float* q_w, const float* k_w, float eps, int rot_dims, int interleaved,
                                      const int32_t* positions, const float* cos_sin, int max_pos, const int64_t* slots, int bs,
                                      void* q_out, void* k_cache, void* v_cache, void* stream) {
     B2_REQUIRE(T >= 0 && H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0 && bs > 0, B2_EINVAL, "qk_rope_cache: bad sizes");
     B2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk, B2_EINVAL,
                "qk_rope_cache: %d rotated entries in heads of %d", rot_dims, dk);
-    B2_REQUIRE(!v_from_k || dv == dk, B2_EINVAL, "qk_rope_cache: values taken from the keys need dv == dk");
+    B2_REQUIRE(Gv > 0 && Gv <= G, B2_EINVAL, "qk_rope_cache: %d value heads beside %d key heads", Gv, G);
+    B2_REQUIRE(!v_from_k || (dv == dk && Gv == G), B2_EINVAL, "qk_rope_cache: values taken from the keys need dv == dk and a value head per key head");
     B2_REQUIRE(rot_dims == 0 || max_pos > 0, B2_EINVAL, "qk_rope_cache: empty rotation table");
     B2_REQUIRE(!q_w == !k_w, B2_EINVAL, "qk_rope_cache: the norm needs the weights of both q and k");
     if (T == 0) return B2_OK;
@@ -837,7 +963,7 @@ extern "C" int b2_qk_norm_rope_cache(const void* qkv, int64_t qkv_stride, int ac
     const int work = (H + G) * dk / (vec ? 4 : 1);
     const int threads = work >= 256 ? 256 : (work >= 128 ? 128 : 64);
 #define B2_ROPE(KERN, NORM)                                                                                                     \
-    KERN<A, NORM><<<T, threads, 0, st>>>(static_cast<const A*>(qkv), qkv_stride, H, G, dk, dv, v_from_k != 0, rot_dims,         \
+    KERN<A, NORM><<<T, threads, 0, st>>>(static_cast<const A*>(qkv), qkv_stride, H, G, Gv, dk, dv, v_from_k != 0, rot_dims,         \
                                          interleaved != 0, positions, cos_sin, max_pos > 0 ? max_pos : 1, slots, bs, q_w, k_w, eps, \
                                          static_cast<A*>(q_out), static_cast<A*>(k_cache), static_cast<A*>(v_cache))
     B2_DISPATCH_ACT(act_dtype, A, {
@@ -856,16 +982,16 @@ extern "C" int b2_chunk_attention(void* out, const void* q, const void* k_cache,
                                   int n_seq, int T, int H, int G, int dk, int dv, int bs, float scale, int chunk, float sink,
                                   float sink_logit, void* stream) {
     return b2_masked_attention(out, q, k_cache, v_cache, act_dtype, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, dk, dv,
-                               bs, scale, chunk, 0, 0, sink, sink_logit, nullptr, B2_WEIGHT_SOFTMAX, nullptr, nullptr, 0,
-                               (int64_t)H * dv, stream);
+                               bs, scale, chunk, 0, 0, sink, sink_logit, nullptr, B2_WEIGHT_SOFTMAX, nullptr, nullptr, 0, 0.f, 1, 0.f,
+                               0.f, 1.f, (int64_t)H * dv, stream);
 }
 
 extern "C" int b2_masked_attention(void* out, const void* q, const void* k_cache, const void* v_cache, int act_dtype,
                                    const int32_t* block_tables, int max_nb, const int32_t* cu_q, const int32_t* ctx_start,
                                    int n_seq, int T, int H, int G, int dk, int dv, int bs, float scale, int chunk, int window,
                                    int keep_first, float sink, float sink_logit, const float* sink_logits, int weight_kind,
-                                   const float* head_bias, const void* gate, int64_t gate_stride, int64_t out_stride,
-                                   void* stream) {
+                                   const float* head_bias, const void* gate, int64_t gate_stride, float softcap, int maps,
+                                   float map_lambda, float map_eps, float map_scale, int64_t out_stride, void* stream) {
     B2_REQUIRE(T >= 0 && H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0 && bs > 0 && chunk >= 0 && sink >= 0.f && window >= 0 &&
                keep_first >= 0, B2_EINVAL, "masked_attention: bad sizes");
     B2_REQUIRE(!gate || gate_stride >= H, B2_EINVAL, "masked_attention: gate rows shorter than the heads");
@@ -874,11 +1000,15 @@ extern "C" int b2_masked_attention(void* out, const void* q, const void* k_cache
     const bool sig = weight_kind == B2_WEIGHT_SIGMOID;
     B2_REQUIRE(sig ? sink == 0.f : !head_bias, B2_EINVAL,
                "masked_attention: sigmoid weights have no sink, and only they take a bias per head");
+    B2_REQUIRE(maps == 1 || maps == 2, B2_EINVAL, "masked_attention: %d maps per head", maps);
+    B2_REQUIRE(!sig || (maps == 1 && softcap == 0.f), B2_EINVAL, "masked_attention: sigmoid weights have one map and no cap");
+    B2_REQUIRE(softcap >= 0.f, B2_EINVAL, "masked_attention: negative cap");
     B2_REQUIRE(out_stride >= (int64_t)H * dv, B2_EINVAL, "masked_attention: output rows shorter than the heads");
     B2_REQUIRE(dv <= 32 * kMaxDvPerLane, B2_EUNSUPPORTED, "chunk_attention: value size %d above %d", dv, 32 * kMaxDvPerLane);
     if (T == 0 || n_seq == 0) return B2_OK;
     B2_REQUIRE(out && q && k_cache && v_cache && block_tables && cu_q && ctx_start, B2_EINVAL, "chunk_attention: null pointer");
     cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const HeadShape hs{softcap, map_lambda, map_eps, map_scale};
     const int warps = 4;
     const size_t smem = (size_t)warps * dk * sizeof(float);
     B2_REQUIRE(smem <= 48 * 1024, B2_EUNSUPPORTED, "chunk_attention: key size %d too large", dk);
@@ -886,47 +1016,55 @@ extern "C" int b2_masked_attention(void* out, const void* q, const void* k_cache
     // prompt chunks of bf16 models with tensor-core friendly head sizes go to the tiled kernel (a sequence needs at least
     // kTileMinRows rows, so a batch of T rows over n_seq sequences can only hold one when T - n_seq >= kTileMinRows - 1)
     int skip_from = 0;
-    if (act_dtype == B2_ACT_BF16 && T - n_seq >= kTileMinRows - 1 && dk % 32 == 0 && dv % 32 == 0 && dk <= 128 && dv <= 128 &&
+    const bool wide = dv == 192 || dv == 256;                // one softmax map only: the accumulators of two would not fit
+    if (act_dtype == B2_ACT_BF16 && T - n_seq >= kTileMinRows - 1 && dk % 32 == 0 && dv % 32 == 0 && dk <= 128 &&
+        (dv <= 128 || (wide && maps == 1 && !sig)) &&
         b2_aligned16(q) && b2_aligned16(k_cache) && b2_aligned16(v_cache) && b2_aligned16(out) && out_stride % 8 == 0) {
         skip_from = kTileMinRows;
         int rc = B2_OK;
+#define B2_TILE_RUN(a, b, SIG, MAPS)                                                                                      \
+    launch_tile<a, b, SIG, MAPS>(q, k_cache, v_cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, bs, scale, chunk, \
+                                 window, keep_first, sink, sink_logit, sink_logits, head_bias, gate, gate_stride, hs, out, \
+                                 out_stride, st)
 #define B2_TILE(a, b)                                                                                                     \
     if (dk == 16 * a && dv == 16 * b)                                                                                     \
-        rc = sig ? launch_tile<a, b, true>(q, k_cache, v_cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, bs, scale, \
-                                           chunk, window, keep_first, 0.f, 0.f, nullptr, head_bias, gate, gate_stride, out,       \
-                                           out_stride, st)                                                                        \
-                 : launch_tile<a, b, false>(q, k_cache, v_cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, bs, scale, \
-                                            chunk, window, keep_first, sink, sink_logit, sink_logits, nullptr, gate, gate_stride, \
-                                            out, out_stride, st);
+        rc = sig ? B2_TILE_RUN(a, b, true, 1) : (maps == 2 ? B2_TILE_RUN(a, b, false, 2) : B2_TILE_RUN(a, b, false, 1));
+#define B2_TILE_WIDE(a, b) if (dk == 16 * a && dv == 16 * b) rc = B2_TILE_RUN(a, b, false, 1);
         B2_TILE(2, 2) B2_TILE(2, 4) B2_TILE(2, 6) B2_TILE(2, 8) B2_TILE(4, 2) B2_TILE(4, 4) B2_TILE(4, 6) B2_TILE(4, 8)
         B2_TILE(6, 2) B2_TILE(6, 4) B2_TILE(6, 6) B2_TILE(6, 8) B2_TILE(8, 2) B2_TILE(8, 4) B2_TILE(8, 6) B2_TILE(8, 8)
+        B2_TILE_WIDE(2, 12) B2_TILE_WIDE(4, 12) B2_TILE_WIDE(6, 12) B2_TILE_WIDE(8, 12)
+        B2_TILE_WIDE(2, 16) B2_TILE_WIDE(4, 16) B2_TILE_WIDE(6, 16) B2_TILE_WIDE(8, 16)
 #undef B2_TILE
+#undef B2_TILE_WIDE
+#undef B2_TILE_RUN
         if (rc != B2_OK) return rc;
     }
     if (act_dtype == B2_ACT_BF16 && dk % 8 == 0 && dv % 8 == 0 && dv <= 64 * kGroupMaxPairs && b2_aligned16(q) &&
         b2_aligned16(k_cache) && b2_aligned16(v_cache) && b2_aligned16(out)) {
         const size_t gsm = (size_t)(kGroupMaxHeads * dk + 4 * kGroupMaxHeads * (2 + dv)) * sizeof(float) +
-                           (size_t)4 * 32 * (dk + 8 + dv) * sizeof(__nv_bfloat16);
-        if (gsm <= 160 * 1024) {
-            auto kern = sig ? chunk_attention_group_kernel<true> : chunk_attention_group_kernel<false>;
+                           (size_t)4 * 32 * (maps * dk + 8 + dv) * sizeof(__nv_bfloat16);
+        if (gsm <= 200 * 1024) {
+            auto kern = sig ? chunk_attention_group_kernel<true, 1>
+                            : (maps == 2 ? chunk_attention_group_kernel<false, 2> : chunk_attention_group_kernel<false, 1>);
             if (gsm > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gsm));
             kern<<<dim3(T, G), 128, gsm, st>>>(static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
                                                static_cast<const __nv_bfloat16*>(v_cache), block_tables, max_nb, cu_q, ctx_start,
                                                n_seq, H, G, dk, dv, bs, scale, chunk, window, keep_first, sink, sink_logit,
-                                               sink_logits, head_bias, static_cast<const __nv_bfloat16*>(gate), gate_stride,
+                                               sink_logits, head_bias, static_cast<const __nv_bfloat16*>(gate), gate_stride, hs,
                                                skip_from, static_cast<__nv_bfloat16*>(out), out_stride);
             B2_CUDA_OK(cudaGetLastError());
             return B2_OK;
         }
     }
-#define B2_WARP_ATTENTION(SIG)                                                                                                \
-    chunk_attention_kernel<A, SIG><<<blocks, warps * 32, smem, st>>>(                                                         \
+#define B2_WARP_ATTENTION(SIG, MAPS)                                                                                          \
+    chunk_attention_kernel<A, SIG, MAPS><<<blocks, warps * 32, smem, st>>>(                                                   \
         static_cast<const A*>(q), static_cast<const A*>(k_cache), static_cast<const A*>(v_cache), block_tables, max_nb, cu_q, \
         ctx_start, n_seq, T, H, G, dk, dv, bs, scale, chunk, window, keep_first, sink, sink_logit, sink_logits, head_bias,    \
-        static_cast<const A*>(gate), gate_stride, skip_from, static_cast<A*>(out), out_stride)
+        static_cast<const A*>(gate), gate_stride, hs, skip_from, static_cast<A*>(out), out_stride)
     B2_DISPATCH_ACT(act_dtype, A, {
-        if (sig) B2_WARP_ATTENTION(true);
-        else B2_WARP_ATTENTION(false);
+        if (sig) B2_WARP_ATTENTION(true, 1);
+        else if (maps == 2) B2_WARP_ATTENTION(false, 2);
+        else B2_WARP_ATTENTION(false, 1);
     });
 #undef B2_WARP_ATTENTION
     B2_CUDA_OK(cudaGetLastError());

@@ -20,7 +20,9 @@
 // number per head (linear attention with a constant decay: S <- lambda_h S + k v^T), the write may be
 // the plain outer product k v^T instead of the delta correction (gated linear attention: S <- diag(decay) S + k v^T),
 // the convolution, its activation and the unit-vector step are optional, and the output gate is SiLU or a sigmoid of
-// a gate row given on its own.  With a decay per channel the decay is applied first: S <- diag(g) S; u = beta (v - S^T k).
+// a gate row given on its own.  q and k heads may be rotated by the token's position (fp32 cos | sin table, either pair
+// layout, the first rot_dims entries) and k scaled, all in fp32 before the scan (retention: a fixed decay per head, rotated
+// q and k, a norm per head without a weight).  With a decay per channel the decay is applied first: S <- diag(g) S; u = beta (v - S^T k).
 //
 // A batch is n sequences; sequence i owns rows cu_q[i] .. cu_q[i+1]-1, has ctx_start[i] tokens before them (< 0: the row
 // group is padding and is skipped) and keeps its state in slot state_slot[i] (< 0: no state is read or written).  A
@@ -46,6 +48,9 @@ struct PrepSpec {
     const float* A_log;      // [H] (softplus modes)
     const float* bias;       // [H] or [H*dk]
     float inv_tau;           // B2_DECAY_CHANNEL_SIGMOID_POW
+    float k_scale;
+    const float* cos_sin;    // [max_pos, rot_dims] = cos | sin halves; rotation of the first rot_dims entries (0: none)
+    int rot_dims, interleaved, max_pos;
 };
 
 template <typename T>
@@ -82,16 +87,29 @@ __global__ void recur_prep_kernel(const T* __restrict__ proj, int64_t proj_strid
     __syncthreads();
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
     float* out = qkv + (size_t)row * C;
+    const float* cs = sp.rot_dims ? sp.cos_sin + (size_t)min(ctx + li, sp.max_pos - 1) * sp.rot_dims : nullptr;
     for (int g = wid; g < 2 * G; g += nw) {          // q heads then k heads
         const float* v = ch + (size_t)g * dk;
-        float sc = g < G ? sp.q_scale : 1.f;
+        float sc = g < G ? sp.q_scale : sp.k_scale;
         if (sp.unit) {
             float ss = 0.f;
             for (int i = lane; i < dk; i += 32) ss = fmaf(v[i], v[i], ss);
             ss = b2::warp_sum(ss);
             sc *= rsqrtf(ss + sp.unit_eps);
         }
-        for (int i = lane; i < dk; i += 32) out[(size_t)g * dk + i] = v[i] * sc;
+        const int half = sp.rot_dims / 2;
+        for (int i = lane; i < dk; i += 32) {
+            float x = v[i];
+            if (i < sp.rot_dims) {
+                int pr, partner;
+                bool second;
+                if (sp.interleaved) { pr = i >> 1; partner = i ^ 1; second = i & 1; }
+                else { second = i >= half; pr = second ? i - half : i; partner = second ? i - half : i + half; }
+                const float c = cs[pr], s = cs[half + pr], other = v[partner];
+                x = second ? fmaf(x, c, other * s) : fmaf(x, c, -other * s);
+            }
+            out[(size_t)g * dk + i] = x * sc;
+        }
     }
     for (int c = 2 * G * dk + threadIdx.x; c < C; c += blockDim.x) out[c] = ch[c];
     const T* pr = proj + (size_t)row * proj_stride;
@@ -420,7 +438,7 @@ __global__ void gated_head_norm_kernel(const float* __restrict__ o, const T* __r
     for (int i = lane; i < dv; i += 32) {
         const float z = b2::ld(g + i);
         const float gv = gate_kind == B2_GATE_SIGMOID ? b2::sigmoid_f(z) : b2::silu_f(z);
-        b2::st(dst + i, ov[i] * inv * norm_w[i] * gv * out_scale);
+        b2::st(dst + i, ov[i] * inv * (norm_w ? norm_w[i] : 1.f) * gv * out_scale);
     }
 }
 
@@ -445,9 +463,9 @@ gated_row_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, i
     const T* g = gate + (size_t)row * gate_stride + (size_t)hh * dv;
     T* dst = out + (size_t)row * out_stride + (size_t)hh * dv;
     for (int i = threadIdx.x * W; i < dv; i += step) {
-        float v[4] = {0.f, 0.f, 0.f, 0.f}, z[4] = {0.f, 0.f, 0.f, 0.f}, w[4] = {0.f, 0.f, 0.f, 0.f};
-        if (W == 4) { b2::ld4(ov + i, v); b2::ld4(g + i, z); b2::ld4(norm_w + i, w); }
-        else { v[0] = ov[i]; z[0] = b2::ld(g + i); w[0] = norm_w[i]; }
+        float v[4] = {0.f, 0.f, 0.f, 0.f}, z[4] = {0.f, 0.f, 0.f, 0.f}, w[4] = {1.f, 1.f, 1.f, 1.f};
+        if (W == 4) { b2::ld4(ov + i, v); b2::ld4(g + i, z); if (norm_w) b2::ld4(norm_w + i, w); }
+        else { v[0] = ov[i]; z[0] = b2::ld(g + i); if (norm_w) w[0] = norm_w[i]; }
 #pragma unroll
         for (int c = 0; c < W; ++c) v[c] *= inv * w[c] * (gate_kind == B2_GATE_SIGMOID ? b2::sigmoid_f(z[c]) : b2::silu_f(z[c]));
         if (W == 4) b2::st4(dst + i, v); else b2::st(dst + i, v[0]);
@@ -539,7 +557,7 @@ extern "C" int b2_delta_prep(const void* proj, int64_t proj_stride, int off_b, i
                "delta_prep: null pointer");
     B2_REQUIRE(conv_state || taps == 1, B2_EINVAL, "delta_prep: a convolution of %d taps needs its state", taps);
     PrepSpec sp{H, G, dk, dv, taps, 1, 1, 1e-6f, 1.f / sqrtf((float)dk), off_b, B2_DECAY_HEAD_SOFTPLUS, off_a, nullptr, 0, A_log,
-                dt_bias, 0.f};
+                dt_bias, 0.f, 1.f, nullptr, 0, 0, 0};
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     int rc = B2_OK;
     B2_DISPATCH_ACT(act_dtype, A, rc = launch_prep<A>(proj, proj_stride, sp, T, conv_w, cu_q, ctx_start, state_slot, n_seq,
@@ -549,7 +567,8 @@ extern "C" int b2_delta_prep(const void* proj, int64_t proj_stride, int off_b, i
 
 extern "C" int b2_recur_prep(const void* proj, int64_t proj_stride, int act_dtype, int T, int H, int G, int dk, int dv,
                              int taps, const float* conv_w, int conv_silu, int unit, float unit_eps, float q_scale,
-                             int off_beta, int decay_mode, int off_a, const float* a, int64_t a_stride, const float* A_log,
+                             float k_scale, const float* cos_sin, int rot_dims, int interleaved, int max_pos, int off_beta,
+                             int decay_mode, int off_a, const float* a, int64_t a_stride, const float* A_log,
                              const float* decay_bias, float tau, const int32_t* cu_q, const int32_t* ctx_start,
                              const int32_t* state_slot, int n_seq, void* conv_state, float* qkv, float* beta, float* decay,
                              void* stream) {
@@ -558,6 +577,8 @@ extern "C" int b2_recur_prep(const void* proj, int64_t proj_stride, int act_dtyp
     B2_REQUIRE(decay_mode == B2_DECAY_HEAD_SOFTPLUS || decay_mode == B2_DECAY_CHANNEL_SOFTPLUS ||
                decay_mode == B2_DECAY_CHANNEL_SIGMOID_POW || decay_mode == B2_DECAY_HEAD_CONST, B2_EINVAL,
                "recur_prep: unknown decay mode %d", decay_mode);
+    B2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || (cos_sin && max_pos > 0)), B2_EINVAL,
+               "recur_prep: %d rotated entries in heads of %d, or no rotation table", rot_dims, dk);
     if (T == 0 || n_seq == 0) return B2_OK;
     B2_REQUIRE(proj && cu_q && ctx_start && state_slot && qkv && decay, B2_EINVAL, "recur_prep: null pointer");
     B2_REQUIRE(conv_w || taps == 1, B2_EINVAL, "recur_prep: a convolution of %d taps needs its weights", taps);
@@ -569,7 +590,8 @@ extern "C" int b2_recur_prep(const void* proj, int64_t proj_stride, int act_dtyp
     if (decay_mode == B2_DECAY_CHANNEL_SOFTPLUS) B2_REQUIRE(A_log, B2_EINVAL, "recur_prep: A_log missing");
     if (decay_mode == B2_DECAY_CHANNEL_SIGMOID_POW) B2_REQUIRE(tau > 0.f, B2_EINVAL, "recur_prep: tau must be positive");
     PrepSpec sp{H, G, dk, dv, taps, conv_silu ? 1 : 0, unit ? 1 : 0, unit_eps, q_scale, off_beta, decay_mode, off_a, a, a_stride,
-                A_log, decay_bias, decay_mode == B2_DECAY_CHANNEL_SIGMOID_POW ? 1.f / tau : 0.f};
+                A_log, decay_bias, decay_mode == B2_DECAY_CHANNEL_SIGMOID_POW ? 1.f / tau : 0.f, k_scale, cos_sin, rot_dims,
+                interleaved ? 1 : 0, max_pos};
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     int rc = B2_OK;
     B2_DISPATCH_ACT(act_dtype, A, rc = launch_prep<A>(proj, proj_stride, sp, T, conv_w, cu_q, ctx_start, state_slot, n_seq,
@@ -612,7 +634,7 @@ extern "C" int b2_gated_head_norm(const float* o, const void* gate, int64_t gate
     B2_REQUIRE(T >= 0 && H > 0 && dv > 0, B2_EINVAL, "gated_head_norm: bad sizes");
     B2_REQUIRE(gate_kind == B2_GATE_SILU || gate_kind == B2_GATE_SIGMOID, B2_EINVAL, "gated_head_norm: unknown gate %d", gate_kind);
     if (T == 0) return B2_OK;
-    B2_REQUIRE(o && gate && norm_w && out, B2_EINVAL, "gated_head_norm: null pointer");
+    B2_REQUIRE(o && gate && out, B2_EINVAL, "gated_head_norm: null pointer");      // norm_w NULL: no weight
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (dv > 512) {                                  // wide rows: a CTA per (row, head) instead of a warp
         const size_t esz = act_dtype == B2_ACT_BF16 ? 2 : 4;

@@ -2,6 +2,9 @@
 // ("hyper-connections"), fused with the pre-norm that follows it:
 //
 //   b2_embed_streams   x[t, s, :] = embed[token[t], :] * scale                      for every stream s
+//   b2_embed_bigram    x[t, :] = embed[token[t], :] + bigram[row, :], row = (token before * mul_prev + token * mul_cur) mod
+//                      buckets in 64-bit integers, or `buckets` (the table's last row) for a sequence's first token.  The token
+//                      before a portion's first row is per-sequence state (one int64 a slot), which the op advances.
 //   b2_hc_step         (1) when y is given: the streams are remixed and the sublayer output is written back,
 //                              x'[t, j, :] = sum_s mix[s, j] * x[t, s, :] + out_w[j] * y[t, :]
 //                      (2) when h is given: the next sublayer's input is read out and normalised,
@@ -26,6 +29,38 @@ __global__ void embed_streams_kernel(const T* __restrict__ embed, const int64_t*
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
         const float v = b2::ld(row + d) * scale;
         for (int s = 0; s < S; ++s) xo[(size_t)s * D + d] = v;
+    }
+}
+
+// The CTA of a portion's first row is the only one that touches the sequence's state: it reads the token before and leaves the
+// portion's last one.
+template <typename T, int W>
+__global__ void embed_bigram_kernel(const T* __restrict__ embed, const T* __restrict__ bigram, const int64_t* __restrict__ tokens,
+                                    int D, int64_t buckets, int64_t mul_prev, int64_t mul_cur, const int32_t* __restrict__ cu_q,
+                                    const int32_t* __restrict__ ctx_start, const int32_t* __restrict__ state_slot, int n_seq,
+                                    int64_t* __restrict__ last_token, float* __restrict__ x) {
+    __shared__ int64_t row_sm;
+    const int t = blockIdx.x;
+    const int64_t tok = tokens[t];
+    if (threadIdx.x == 0) {
+        const int seq = b2::seq_of_row(cu_q, n_seq, t);
+        const int r0 = cu_q[seq], ctx = ctx_start[seq], slot = ctx >= 0 ? state_slot[seq] : -1;
+        int64_t prev = -1;                           // none: the sequence's first token
+        if (t > r0) prev = tokens[t - 1];
+        else if (ctx > 0 && slot >= 0) prev = last_token[slot];
+        if (t == r0 && slot >= 0) last_token[slot] = tokens[cu_q[seq + 1] - 1];
+        row_sm = prev < 0 ? buckets : (prev * mul_prev + tok * mul_cur) % buckets;
+    }
+    __syncthreads();
+    const T* a = embed + (size_t)tok * D;
+    const T* b = bigram + (size_t)row_sm * D;
+    float* xo = x + (size_t)t * D;
+    for (int d = threadIdx.x * W; d < D; d += blockDim.x * W) {
+        float u[4] = {0.f, 0.f, 0.f, 0.f}, v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (W == 4) { b2::ld4(a + d, u); b2::ld4(b + d, v); } else { u[0] = b2::ld(a + d); v[0] = b2::ld(b + d); }
+#pragma unroll
+        for (int c = 0; c < W; ++c) u[c] += v[c];
+        if (W == 4) b2::st4(xo + d, u); else xo[d] = u[0];
     }
 }
 
@@ -126,6 +161,26 @@ extern "C" int b2_embed_streams(float* x, const void* embed, int act_dtype, cons
     B2_REQUIRE(x && embed && tokens, B2_EINVAL, "embed_streams: null pointer");
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     B2_DISPATCH_ACT(act_dtype, A, (embed_streams_kernel<A><<<T, 256, 0, st>>>(static_cast<const A*>(embed), tokens, D, S, scale, x)));
+    B2_CUDA_OK(cudaGetLastError());
+    return B2_OK;
+}
+
+extern "C" int b2_embed_bigram(float* x, const void* embed, const void* bigram, int act_dtype, const int64_t* tokens, int T, int D,
+                               int64_t buckets, int64_t mul_prev, int64_t mul_cur, const int32_t* cu_q, const int32_t* ctx_start,
+                               const int32_t* state_slot, int n_seq, int64_t* last_token, void* stream) {
+    B2_REQUIRE(T >= 0 && D > 0 && buckets > 0 && mul_prev >= 0 && mul_cur >= 0, B2_EINVAL, "embed_bigram: bad sizes T=%d D=%d", T, D);
+    if (T == 0 || n_seq == 0) return B2_OK;
+    B2_REQUIRE(x && embed && bigram && tokens && cu_q && ctx_start && state_slot && last_token, B2_EINVAL, "embed_bigram: null pointer");
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const bool vec = D % 4 == 0 && b2_aligned16(x) && b2_aligned16(embed) && b2_aligned16(bigram);
+#define B2_BIGRAM(W)                                                                                                        \
+    embed_bigram_kernel<A, W><<<T, 256, 0, st>>>(static_cast<const A*>(embed), static_cast<const A*>(bigram), tokens, D, buckets,  \
+                                                 mul_prev, mul_cur, cu_q, ctx_start, state_slot, n_seq, last_token, x)
+    B2_DISPATCH_ACT(act_dtype, A, {
+        if (vec) B2_BIGRAM(4);
+        else B2_BIGRAM(1);
+    });
+#undef B2_BIGRAM
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }

@@ -6,7 +6,8 @@
 //                    B2_ROUTE_SIGMOID_GROUPED: s = sigmoid(z); the choice looks at c = s + b; the experts form `n_groups` equal
 //                    groups of neighbours, a group's score is the sum of its two largest c, and only experts of the
 //                    `keep_groups` best groups can be chosen (the others count as -inf); weights = the chosen s divided by
-//                    their sum (+ 1e-20), times `weight_scale`.  (b2_moe_route_ex / b2_moe_select_ex carry the three
+//                    their sum (+ 1e-20), times `weight_scale`.  B2_ROUTE_SIGMOID_PLAIN: the same choice, weights = the chosen
+//                    s times `weight_scale`, not divided by their sum.  (b2_moe_route_ex / b2_moe_select_ex carry the three
 //                    parameters; n_groups = 1 is the ungrouped case.)
 //   b2_moe_select    the same choice from fp32 logits computed elsewhere (a library GEMM over a prompt batch).
 //   b2_moe_align     counting sort of the T*top (token, choice) pairs by expert into row tiles of kMoeBM rows: every tile
@@ -17,8 +18,12 @@
 //                    g' * sigmoid(alpha * g') * (u' + 1) (B2_GLU_CLAMPED).  B2_FF_RELU_SQ: experts without a gate,
 //                    act = max(h W_up[e]^T, 0)^2 (w_gate is not read).
 //   b2_moe_down      per tile: rows = act W_down[e]^T, fp32.
-//   b2_moe_combine   y[t] = sum_j weight[t, j] * rows[place of (t, j)], summed in choice order in fp32: a token's result
-//                    does not depend on what else is in the batch.
+//   b2_moe_combine   y[t] = (add[t] +) sum_j weight[t, j] * rows[place of (t, j)], summed in choice order in fp32: a token's
+//                    result does not depend on what else is in the batch.  `add` is the output of an expert that every token
+//                    uses.
+// A design may weight an expert's INPUT instead of its output, y = sum_j expert_j(weight_j * h) (b2_moe_experts with
+// weight_on_input): both first products are linear in h, so the weight multiplies their fp32 accumulators before the
+// activation, and the sum at the end takes the rows as they are.  (b2_moe_gather with weights scales the gathered rows.)
 // The two grouped products are tiled through shared memory; bf16 runs on the tensor cores (16x16x16 fragments, fp32
 // accumulation), the all-32-bit mode on fp32 FMAs.  Expert weights are stacked: w_gate, w_up [E, F, D]; w_down [E, D, F].
 #include "b2_act.cuh"
@@ -38,7 +43,8 @@ struct RouteSpec {
 };
 
 // floats of scratch per token beside its E logits
-__host__ __device__ __forceinline__ int route_scratch(int scoring, int E) { return scoring == B2_ROUTE_SIGMOID_GROUPED ? 2 * E : 0; }
+__host__ __device__ __forceinline__ bool route_sigmoid(int scoring) { return scoring == B2_ROUTE_SIGMOID_GROUPED || scoring == B2_ROUTE_SIGMOID_PLAIN; }
+__host__ __device__ __forceinline__ int route_scratch(int scoring, int E) { return route_sigmoid(scoring) ? 2 * E : 0; }
 
 // lowest index wins a tie; every lane returns the winner
 __device__ __forceinline__ int warp_argmax(const float* c, int E, int lane, float& best_out) {
@@ -59,7 +65,7 @@ __device__ __forceinline__ int warp_argmax(const float* c, int E, int lane, floa
 __device__ __forceinline__ void route_select(float* z, int t, int E, int top, RouteSpec rs, const float* __restrict__ bias,
                                              int lane, int32_t* __restrict__ ids, float* __restrict__ wts) {
     const int scoring = rs.scoring;
-    if (scoring == B2_ROUTE_SIGMOID_GROUPED) {
+    if (route_sigmoid(scoring)) {
         float* c = z + E;                            // choice scores; then the group scores
         float* gs = z + 2 * E;
         for (int e = lane; e < E; e += 32) {
@@ -101,7 +107,7 @@ __device__ __forceinline__ void route_select(float* z, int t, int E, int top, Ro
             }
             __syncwarp();
         }
-        const float inv = rs.weight_scale / (sum + 1e-20f);
+        const float inv = scoring == B2_ROUTE_SIGMOID_PLAIN ? rs.weight_scale : rs.weight_scale / (sum + 1e-20f);
         for (int j = lane; j < top; j += 32) wts[(size_t)t * top + j] *= inv;
         return;
     }
@@ -478,7 +484,8 @@ template <typename T, int NB>
 __global__ void __launch_bounds__(128)
 moe_gate_up_kernel(const T* __restrict__ h, int64_t h_stride, const T* __restrict__ w_gate, const T* __restrict__ w_up,
                    int64_t w13_expert_stride, const int32_t* __restrict__ sorted, const int32_t* __restrict__ tile_expert,
-                   int top, int D, int F, bool vec, int glu, float alpha, float limit, T* __restrict__ act) {
+                   int top, int D, int F, bool vec, int glu, float alpha, float limit, const float* __restrict__ in_w,
+                   T* __restrict__ act) {
     __shared__ __align__(128) unsigned char sm[TileSmem<T, NB>::BYTES];
     const float* c_sm = reinterpret_cast<const float*>(sm);
     const int e = tile_expert[blockIdx.x];
@@ -496,12 +503,14 @@ moe_gate_up_kernel(const T* __restrict__ h, int64_t h_stride, const T* __restric
     else tile_product<T, NB>(a_row, u_row, u_row, D, vec, sm);
     for (int idx = threadIdx.x; idx < kMoeBM * kMoeBN; idx += blockDim.x) {
         const int r = idx / kMoeBN, c = idx % kMoeBN;
-        if (n0 + c < F && sorted[m0 + r] >= 0) {
+        const int pair = sorted[m0 + r];
+        if (n0 + c < F && pair >= 0) {
+            const float wt = in_w ? in_w[pair] : 1.f;           // weight on the expert's input: W (wt h) = wt (W h)
             float v;
             if (NB == 1) {
-                v = b2::relu_sq_f(c_sm[idx]);
+                v = b2::relu_sq_f(wt * c_sm[idx]);
             } else {
-                const float g = c_sm[idx], u = c_sm[(NB - 1) * kMoeBM * kMoeBN + idx];
+                const float g = wt * c_sm[idx], u = wt * c_sm[(NB - 1) * kMoeBM * kMoeBN + idx];
                 v = glu == B2_GLU_CLAMPED ? b2::glu_clamped_f(g, u, alpha, limit) : b2::silu_f(g) * u;
             }
             b2::st(act + (size_t)(m0 + r) * F + n0 + c, v);
@@ -528,14 +537,27 @@ moe_down_kernel(const T* __restrict__ act, const T* __restrict__ w_down, const i
     }
 }
 
-// out[p] = h[token of sorted[p]] for the rows of the sorted list, zeros for padding rows: the A operand of a grouped GEMM
+// out[p] = h[token of sorted[p]] (times the pair's weight when given) for the rows of the sorted list, zeros for padding rows: the A operand of a grouped GEMM
 template <typename T>
 __global__ void moe_gather_kernel(const T* __restrict__ h, int64_t h_stride, const int32_t* __restrict__ sorted, int top,
-                                  int D, bool vec, T* __restrict__ out) {
+                                  int D, bool vec, const float* __restrict__ wts, T* __restrict__ out) {
     const int p = blockIdx.x, s = sorted[p];
+    const float wt = wts && s >= 0 ? wts[s] : 1.f;
     const T* src = s >= 0 ? h + (size_t)(s / top) * h_stride : nullptr;
     T* dst = out + (size_t)p * D;
-    if (vec) {
+    if (wts) {
+        if (vec) {
+            for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                if (src) b2::ld4(src + i, v);
+#pragma unroll
+                for (int c = 0; c < 4; ++c) v[c] *= wt;
+                b2::st4(dst + i, v);
+            }
+        } else {
+            for (int i = threadIdx.x; i < D; i += blockDim.x) b2::st(dst + i, src ? wt * b2::ld(src + i) : 0.f);
+        }
+    } else if (vec) {
         constexpr int VE = 16 / sizeof(T);
         for (int i = threadIdx.x * VE; i < D; i += blockDim.x * VE)
             *reinterpret_cast<uint4*>(dst + i) = src ? *reinterpret_cast<const uint4*>(src + i) : make_uint4(0, 0, 0, 0);
@@ -544,18 +566,42 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, int64_t h_stride, con
     }
 }
 
-template <typename T, typename R>
+template <typename T, typename R, int W>
 __global__ void moe_combine_kernel(const R* __restrict__ rows, const int32_t* __restrict__ place,
-                                   const float* __restrict__ wts, int top, int D, T* __restrict__ y, int64_t y_stride) {
+                                   const float* __restrict__ wts, int top, int D, const T* __restrict__ add, int64_t add_stride,
+                                   T* __restrict__ y, int64_t y_stride) {
     const int t = blockIdx.x;
-    for (int d = threadIdx.x; d < D; d += blockDim.x) {
-        float a = 0.f;
+    for (int d = threadIdx.x * W; d < D; d += blockDim.x * W) {
+        float a[4] = {0.f, 0.f, 0.f, 0.f};
+        if (add) {
+            if (W == 4) b2::ld4(add + (size_t)t * add_stride + d, a); else a[0] = b2::ld(add + (size_t)t * add_stride + d);
+        }
         for (int j = 0; j < top; ++j) {
             const int p = place[(size_t)t * top + j];
-            if (p >= 0) a = fmaf(wts[(size_t)t * top + j], b2::ld(rows + (size_t)p * D + d), a);
+            if (p < 0) continue;
+            const float wt = wts ? wts[(size_t)t * top + j] : 1.f;
+            float v[4] = {0.f, 0.f, 0.f, 0.f};
+            if (W == 4) b2::ld4(rows + (size_t)p * D + d, v); else v[0] = b2::ld(rows + (size_t)p * D + d);
+#pragma unroll
+            for (int c = 0; c < W; ++c) a[c] = fmaf(wt, v[c], a[c]);
         }
-        b2::st(y + (size_t)t * y_stride + d, a);
+        if (W == 4) b2::st4(y + (size_t)t * y_stride + d, a); else b2::st(y + (size_t)t * y_stride + d, a[0]);
     }
+}
+
+template <typename T, typename R>
+int launch_combine(const void* rows, const int32_t* place, const float* wts, int rows_n, int top, int D, const void* add,
+                   int64_t add_stride, void* y, int64_t y_stride, cudaStream_t st) {
+    const bool vec = D % 4 == 0 && y_stride % 4 == 0 && b2_aligned16(rows) && b2_aligned16(y) &&
+                     (!add || (add_stride % 4 == 0 && b2_aligned16(add)));
+    if (vec)
+        moe_combine_kernel<T, R, 4><<<rows_n, 256, 0, st>>>(static_cast<const R*>(rows), place, wts, top, D, static_cast<const T*>(add),
+                                                           add_stride, static_cast<T*>(y), y_stride);
+    else
+        moe_combine_kernel<T, R, 1><<<rows_n, 256, 0, st>>>(static_cast<const R*>(rows), place, wts, top, D, static_cast<const T*>(add),
+                                                           add_stride, static_cast<T*>(y), y_stride);
+    B2_CUDA_OK(cudaGetLastError());
+    return B2_OK;
 }
 
 }  // namespace
@@ -570,7 +616,7 @@ extern "C" int b2_moe_capacity(int n, int E) {
 
 static bool route_spec_ok(int scoring, int E, int top, int n_groups, int keep_groups) {
     if (scoring == B2_ROUTE_TOPK_SOFTMAX || scoring == B2_ROUTE_SOFTMAX_ALL) return true;
-    if (scoring != B2_ROUTE_SIGMOID_GROUPED) return false;
+    if (!route_sigmoid(scoring)) return false;
     return n_groups >= 1 && E % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups &&
            (int64_t)keep_groups * (E / n_groups) >= top;
 }
@@ -656,7 +702,8 @@ extern "C" int b2_moe_experts(const void* h, int64_t h_stride, const void* w_gat
                               int64_t w13_expert_stride, int act_dtype, int T, int D, int F, int top, int cap,
                               const int32_t* sorted,
                               const int32_t* tile_expert, const int32_t* place, const float* weights, void* act, float* rows,
-                              void* y, int64_t y_stride, int glu, float glu_alpha, float glu_limit, void* stream) {
+                              const void* add, int64_t add_stride, void* y, int64_t y_stride, int glu, float glu_alpha,
+                              float glu_limit, int weight_on_input, void* stream) {
     B2_REQUIRE(T >= 0 && D > 0 && F > 0 && top >= 1 && cap % kMoeBM == 0, B2_EINVAL, "moe_experts: bad sizes");
     B2_REQUIRE(glu == B2_GLU_SILU || glu == B2_GLU_CLAMPED || glu == B2_FF_RELU_SQ, B2_EINVAL,
                "moe_experts: unknown expert activation %d", glu);
@@ -668,6 +715,8 @@ extern "C" int b2_moe_experts(const void* h, int64_t h_stride, const void* w_gat
     const int tiles = cap / kMoeBM;
     const int ve = act_dtype == B2_ACT_BF16 ? 8 : 4;
     B2_REQUIRE(w13_expert_stride >= (int64_t)F * D, B2_EINVAL, "moe_experts: expert stride below F*D");
+    const float* in_w = weight_on_input ? weights : nullptr;
+    int rc = B2_OK;
     const bool vec1 = D % ve == 0 && h_stride % ve == 0 && w13_expert_stride % ve == 0 && b2_aligned16(h) &&
                       (!gated || b2_aligned16(w_gate)) && b2_aligned16(w_up);
     const bool vec2 = F % ve == 0 && b2_aligned16(act) && b2_aligned16(w_down);
@@ -675,21 +724,22 @@ extern "C" int b2_moe_experts(const void* h, int64_t h_stride, const void* w_gat
         if (gated)
             moe_gate_up_kernel<A, 2><<<dim3(tiles, (F + kMoeBN - 1) / kMoeBN), 128, 0, st>>>(
                 static_cast<const A*>(h), h_stride, static_cast<const A*>(w_gate), static_cast<const A*>(w_up), w13_expert_stride,
-                sorted, tile_expert, top, D, F, vec1, glu, glu_alpha, glu_limit, static_cast<A*>(act));
+                sorted, tile_expert, top, D, F, vec1, glu, glu_alpha, glu_limit, in_w, static_cast<A*>(act));
         else
             moe_gate_up_kernel<A, 1><<<dim3(tiles, (F + kMoeBN - 1) / kMoeBN), 128, 0, st>>>(
                 static_cast<const A*>(h), h_stride, nullptr, static_cast<const A*>(w_up), w13_expert_stride, sorted, tile_expert,
-                top, D, F, vec1, glu, glu_alpha, glu_limit, static_cast<A*>(act));
+                top, D, F, vec1, glu, glu_alpha, glu_limit, in_w, static_cast<A*>(act));
         moe_down_kernel<A><<<dim3(tiles, (D + kMoeBN - 1) / kMoeBN), 128, 0, st>>>(
             static_cast<const A*>(act), static_cast<const A*>(w_down), sorted, tile_expert, D, F, vec2, rows);
-        moe_combine_kernel<A, float><<<T, 256, 0, st>>>(rows, place, weights, top, D, static_cast<A*>(y), y_stride);
+        rc = launch_combine<A, float>(rows, place, weight_on_input ? nullptr : weights, T, top, D, add, add_stride, y, y_stride, st);
     });
+    if (rc != B2_OK) return rc;
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }
 
-extern "C" int b2_moe_gather(const void* h, int64_t h_stride, int act_dtype, const int32_t* sorted, int cap, int top, int D,
-                             void* out, void* stream) {
+extern "C" int b2_moe_gather(const void* h, int64_t h_stride, int act_dtype, const int32_t* sorted, const float* weights, int cap,
+                             int top, int D, void* out, void* stream) {
     B2_REQUIRE(cap >= 0 && top >= 1 && D > 0, B2_EINVAL, "moe_gather: bad sizes");
     if (cap == 0) return B2_OK;
     B2_REQUIRE(h && sorted && out, B2_EINVAL, "moe_gather: null pointer");
@@ -697,24 +747,23 @@ extern "C" int b2_moe_gather(const void* h, int64_t h_stride, int act_dtype, con
     const bool vec = D % ve == 0 && h_stride % ve == 0 && b2_aligned16(h) && b2_aligned16(out);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     B2_DISPATCH_ACT(act_dtype, A, (moe_gather_kernel<A><<<cap, 128, 0, st>>>(static_cast<const A*>(h), h_stride, sorted, top, D, vec,
-                                                                           static_cast<A*>(out))));
+                                                                           weights, static_cast<A*>(out))));
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
 }
 
-// y[t] = sum_j weights[t, j] * rows[place[t, j]] in fp32, choice order; rows in the activation type (rows_f32 = 0) or fp32
+// y[t] = (add[t] +) sum_j weights[t, j] * rows[place[t, j]] in fp32, choice order (weights NULL: ones); rows in the activation
+// type (rows_f32 = 0) or fp32
 extern "C" int b2_moe_combine(const void* rows, int rows_f32, const int32_t* place, const float* weights, int T, int top, int D,
-                              void* y, int64_t y_stride, int act_dtype, void* stream) {
+                              const void* add, int64_t add_stride, void* y, int64_t y_stride, int act_dtype, void* stream) {
     B2_REQUIRE(T >= 0 && top >= 1 && D > 0, B2_EINVAL, "moe_combine: bad sizes");
     if (T == 0) return B2_OK;
-    B2_REQUIRE(rows && place && weights && y, B2_EINVAL, "moe_combine: null pointer");
+    B2_REQUIRE(rows && place && y, B2_EINVAL, "moe_combine: null pointer");
     cudaStream_t st = static_cast<cudaStream_t>(stream);
+    int rc = B2_OK;
     B2_DISPATCH_ACT(act_dtype, A, {
-        if (rows_f32) moe_combine_kernel<A, float><<<T, 256, 0, st>>>(static_cast<const float*>(rows), place, weights, top, D,
-                                                                      static_cast<A*>(y), y_stride);
-        else moe_combine_kernel<A, A><<<T, 256, 0, st>>>(static_cast<const A*>(rows), place, weights, top, D, static_cast<A*>(y),
-                                                         y_stride);
+        if (rows_f32) rc = launch_combine<A, float>(rows, place, weights, T, top, D, add, add_stride, y, y_stride, st);
+        else rc = launch_combine<A, A>(rows, place, weights, T, top, D, add, add_stride, y, y_stride, st);
     });
-    B2_CUDA_OK(cudaGetLastError());
-    return B2_OK;
+    return rc;
 }

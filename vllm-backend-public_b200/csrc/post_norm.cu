@@ -8,6 +8,9 @@
 //                      norm = layer norm (B2_NORM_LAYER, bias optional) or RMS norm (B2_NORM_RMS), eps inside the root.
 //                      The write-back and the next read-out touch the same row, so the op moves D*4 in, D*4 out for the
 //                      residual plus one activation row each way.  With post_w = NULL it is residual add + pre-norm.
+//   b2_sandwich_norm_pair   the same with the sublayer output made of two rows side by side, each normalised first:
+//                      y = scale * (norm(y1; w1) + norm(y2; w2)) -- a mixer of two halves -- in fp32 from the halves' rows to the
+//                      residual, three norms and the sum in one pass.
 //   b2_row_norm        out[t, :] = in[t, :] / sqrt(mean(in[t, :]^2) + eps) * w over activation rows of any width (row strides
 //                      of their own: a column range of a wider projection is fine); the statistics in fp32.  The norm of a
 //                      low-rank latent between its two projections.
@@ -29,12 +32,21 @@ namespace {
 
 // W = 4: every access is a 16-byte (fp32) or 8-byte (bf16) vector; W = 1: any width and alignment.  A thread keeps to its
 // own columns in every pass, so the row in shared memory needs no barrier beyond those of the reductions.
-template <typename T, int W>
+// A sublayer output in two halves (see b2_sandwich_norm_pair).
+template <typename T>
+struct PairRows {
+    const T* y2;
+    int64_t y2_stride;
+    const float *w1, *w2;
+    float scale;
+};
+
+template <typename T, int W, bool PAIR>
 __global__ void __launch_bounds__(512)
-sandwich_norm_kernel(float* __restrict__ x, int D, const T* __restrict__ y, int64_t y_stride, const float* __restrict__ post_w,
+sandwich_norm_kernel(float* __restrict__ x, int D, const T* __restrict__ y, int64_t y_stride, PairRows<T> pair, const float* __restrict__ post_w,
                      const float* __restrict__ post_b, const float* __restrict__ pre_w, const float* __restrict__ pre_b, float eps,
                      int norm_kind, T* __restrict__ h, int64_t h_stride) {
-    extern __shared__ __align__(16) float row_sm[];  // [D]
+    extern __shared__ __align__(16) float row_sm[];  // [D], PAIR: [2 D]
     __shared__ float red[33];
     const int t = blockIdx.x;
     float* xt = x + (size_t)t * D;
@@ -49,6 +61,31 @@ sandwich_norm_kernel(float* __restrict__ x, int D, const T* __restrict__ y, int6
             for (int c = 0; c < W; ++c) {
                 row_sm[d + c] = v[c];
                 sum += v[c];
+            }
+        }
+        if (PAIR) {                                  // both halves' own norms, then their scaled sum takes the row's place
+            const T* y2 = pair.y2 + (size_t)t * pair.y2_stride;
+            float s1 = 0.f, s2 = 0.f;
+            for (int d = threadIdx.x * W; d < D; d += step) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                if (W == 4) b2::ld4(y2 + d, v); else v[0] = b2::ld(y2 + d);
+#pragma unroll
+                for (int c = 0; c < W; ++c) {
+                    row_sm[D + d + c] = v[c];
+                    s2 = fmaf(v[c], v[c], s2);
+                    s1 = fmaf(row_sm[d + c], row_sm[d + c], s1);
+                }
+            }
+            const float i1 = rsqrtf(b2::block_sum(s1, red) / (float)D + eps) * pair.scale;
+            const float i2 = rsqrtf(b2::block_sum(s2, red) / (float)D + eps) * pair.scale;
+            sum = 0.f;
+            for (int d = threadIdx.x * W; d < D; d += step) {
+#pragma unroll
+                for (int c = 0; c < W; ++c) {
+                    const float v = row_sm[d + c] * i1 * pair.w1[d + c] + row_sm[D + d + c] * i2 * pair.w2[d + c];
+                    row_sm[d + c] = v;
+                    sum += v;
+                }
             }
         }
         float mean = 0.f, inv = 1.f;
@@ -278,34 +315,53 @@ inline dim3 rows_grid(int cols, int rows) {
 
 }  // namespace
 
-extern "C" int b2_sandwich_norm(float* x, int T, int D, const void* y, int64_t y_stride, const float* post_w,
-                                const float* post_b, const float* pre_w, const float* pre_b, float eps, int norm_kind, void* h,
-                                int64_t h_stride, int act_dtype, void* stream) {
+static int sandwich_norm(float* x, int T, int D, const void* y, int64_t y_stride, const void* y2, int64_t y2_stride, const float* w1,
+                         const float* w2, float pair_scale, const float* post_w, const float* post_b, const float* pre_w,
+                         const float* pre_b, float eps, int norm_kind, void* h, int64_t h_stride, int act_dtype, void* stream) {
     B2_REQUIRE(T >= 0 && D > 0, B2_EINVAL, "sandwich_norm: bad sizes T=%d D=%d", T, D);
     if (T == 0 || (!y && !h)) return B2_OK;
     B2_REQUIRE(x, B2_EINVAL, "sandwich_norm: null residual");
     B2_REQUIRE(!h || pre_w, B2_EINVAL, "sandwich_norm: a read-out needs its norm weight");
     B2_REQUIRE(norm_kind == B2_NORM_LAYER || norm_kind == B2_NORM_RMS, B2_EINVAL, "sandwich_norm: unknown norm kind %d", norm_kind);
-    const size_t smem = (size_t)D * sizeof(float);
+    const size_t smem = (size_t)(y2 ? 2 : 1) * D * sizeof(float);
     B2_REQUIRE(smem <= 200 * 1024, B2_EUNSUPPORTED, "sandwich_norm: width %d does not fit shared memory", D);
     B2_REQUIRE(b2_aligned16(x), B2_EINVAL, "sandwich_norm: the residual must be 16-byte aligned");
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     const int threads = D >= 8192 ? 512 : (D >= 1024 ? 256 : 128);
-    const bool vec = D % 4 == 0 && (!y || (y_stride % 4 == 0 && b2_aligned16(y))) && (!h || (h_stride % 4 == 0 && b2_aligned16(h)));
-#define B2_SANDWICH(W)                                                                                                      \
+    const bool vec = D % 4 == 0 && (!y || (y_stride % 4 == 0 && b2_aligned16(y))) && (!h || (h_stride % 4 == 0 && b2_aligned16(h))) &&
+                     (!y2 || (y2_stride % 4 == 0 && b2_aligned16(y2)));
+#define B2_SANDWICH(W, PAIR)                                                                                                \
     do {                                                                                                                    \
-        auto kern = sandwich_norm_kernel<A, W>;                                                                             \
+        auto kern = sandwich_norm_kernel<A, W, PAIR>;                                                                       \
         if (smem > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-        kern<<<T, threads, smem, st>>>(x, D, static_cast<const A*>(y), y_stride, post_w, post_b, pre_w, pre_b, eps, norm_kind, \
-                                       static_cast<A*>(h), h_stride);                                                       \
+        kern<<<T, threads, smem, st>>>(x, D, static_cast<const A*>(y), y_stride,                                            \
+                                       PairRows<A>{static_cast<const A*>(y2), y2_stride, w1, w2, pair_scale}, post_w, post_b, pre_w, \
+                                       pre_b, eps, norm_kind, static_cast<A*>(h), h_stride);                                \
     } while (0)
     B2_DISPATCH_ACT(act_dtype, A, {
-        if (vec) B2_SANDWICH(4);
-        else B2_SANDWICH(1);
+        if (y2 && vec) B2_SANDWICH(4, true);
+        else if (y2) B2_SANDWICH(1, true);
+        else if (vec) B2_SANDWICH(4, false);
+        else B2_SANDWICH(1, false);
     });
 #undef B2_SANDWICH
     B2_CUDA_OK(cudaGetLastError());
     return B2_OK;
+}
+
+extern "C" int b2_sandwich_norm(float* x, int T, int D, const void* y, int64_t y_stride, const float* post_w,
+                                const float* post_b, const float* pre_w, const float* pre_b, float eps, int norm_kind, void* h,
+                                int64_t h_stride, int act_dtype, void* stream) {
+    return sandwich_norm(x, T, D, y, y_stride, nullptr, 0, nullptr, nullptr, 1.f, post_w, post_b, pre_w, pre_b, eps, norm_kind, h,
+                         h_stride, act_dtype, stream);
+}
+
+extern "C" int b2_sandwich_norm_pair(float* x, int T, int D, const void* y1, int64_t y1_stride, const float* w1, const void* y2,
+                                     int64_t y2_stride, const float* w2, float pair_scale, const float* post_w, const float* pre_w,
+                                     float eps, void* h, int64_t h_stride, int act_dtype, void* stream) {
+    B2_REQUIRE(y1 && y2 && w1 && w2, B2_EINVAL, "sandwich_norm_pair: both rows and their weights are needed");
+    return sandwich_norm(x, T, D, y1, y1_stride, y2, y2_stride, w1, w2, pair_scale, post_w, nullptr, pre_w, nullptr, eps, B2_NORM_RMS, h,
+                         h_stride, act_dtype, stream);
 }
 
 extern "C" int b2_row_norm(void* out, int64_t out_stride, const void* in, int64_t in_stride, int act_dtype, int T, int n,
