@@ -13,7 +13,6 @@ from that config.json.  head_dim must be 128 (what the attention kernels are bui
 from __future__ import annotations
 
 import json
-import math
 import os
 from dataclasses import dataclass, field
 from pathlib import Path
@@ -133,13 +132,8 @@ def rope_table(max_pos: int, d: int, theta: float, scaling: Optional[dict], devi
     Same construction as the oracle's table (oracle/layer_ref.py::rope_table); transformers' llama3 init agrees."""
     inv = 1.0 / (theta ** (torch.arange(0, d, 2, dtype=torch.float64) / d))
     if scaling:
-        f, lo, hi = scaling["factor"], scaling["low_freq_factor"], scaling["high_freq_factor"]
-        old = scaling["original_max_position_embeddings"]
-        wavelen = 2 * math.pi / inv
-        smooth = ((old / wavelen) - lo) / (hi - lo)
-        scaled = torch.where(wavelen > old / lo, inv / f, inv)
-        mid = (wavelen <= old / lo) & (wavelen >= old / hi)
-        inv = torch.where(mid, (1 - smooth) * inv / f + smooth * inv, scaled)
+        inv = ops.three_zone_frequencies(inv, scaling["factor"], scaling["low_freq_factor"], scaling["high_freq_factor"],
+                                         scaling["original_max_position_embeddings"])
     ang = torch.arange(max_pos, dtype=torch.float64).unsqueeze(1) * inv.unsqueeze(0)
     return torch.cat([torch.cos(ang), torch.sin(ang)], dim=1).to(torch.float32).contiguous().to(device)
 
@@ -406,12 +400,13 @@ class LlamaModel:
 
 
 def _register_families() -> None:
-    from . import gapidra, gatolix, kofadra, sanarax, tonilix
+    from . import gapidra, gatolix, kofadra, lizazen, sanarax, tonilix
     ARCHITECTURES[kofadra.ARCHITECTURE] = kofadra.config_from_dir
     ARCHITECTURES[gatolix.ARCHITECTURE] = gatolix.config_from_dir
     ARCHITECTURES[tonilix.ARCHITECTURE] = tonilix.config_from_dir
     ARCHITECTURES[sanarax.ARCHITECTURE] = sanarax.config_from_dir
     ARCHITECTURES[gapidra.ARCHITECTURE] = gapidra.config_from_dir
+    ARCHITECTURES[lizazen.ARCHITECTURE] = lizazen.config_from_dir
 
 
 _register_families()
