@@ -32,10 +32,11 @@
 //   b2_qk_norm_rope_cache  rows [q | k | v]: all of q (H * dk numbers) and all of k (G * dk) are RMS-normed as one row each,
 //                        before the split into heads (fp32 weights of those sizes), then rotated and written as above; the
 //                        numbers stay in fp32 between the norm and the rotation.
-//   b2_chunk_attention   per (token, head) one warp: scores of 32 keys at a time (a lane per key), online softmax in fp32
-//                        seeded with the sink, P.V with a lane per value column.  With the mask a query touches at most
-//                        `chunk` keys wherever it stands, so prompt chunks and decode rows run the same kernel; a decode
-//                        row is a sequence with one query.
+//   b2_chunk_attention   four kernels: prompt rows of bf16 models on mma.sync tiles of 64 rows; decode rows and short portions
+//                        of bf16 models on mma.sync with a kv head's query heads as operand rows, or (head sizes the tensor
+//                        cores do not take) one CTA per (row, kv head) on fp32 FMAs; fp32 and odd sizes one warp per
+//                        (token, head).  Scores, softmax state and accumulators are fp32 in all of them.  With a mask a query
+//                        touches only the keys it sees, wherever it stands; a decode row is a sequence with one query.
 // Sequences are described like everywhere in this library: rows cu_q[i] .. cu_q[i+1]-1, ctx_start[i] cached tokens
 // before them (< 0: padding, output rows are zeroed), block_tables[i, :].
 #include "b2_act.cuh"
@@ -369,7 +370,7 @@ __global__ void chunk_attention_kernel(const T* __restrict__ q, const T* __restr
 }
 
 // ------------------------------------------------------------------------------------------------- grouped decode kernel
-// bf16 rows that the tiled kernel does not take (decode rows, short portions): one CTA per (row, kv head) serves ALL the
+// bf16 rows that neither tensor-core kernel takes (decode rows and short portions of other head sizes): one CTA per (row, kv head) serves ALL the
 // query heads of that kv head, so K and V are read once per group instead of once per head.  Four warps share the visible
 // keys 32 at a time (a lane per key, 16-byte loads of its K row, one dot product per query head), keep an online softmax
 // per head, accumulate P.V with a lane per pair of value columns, and merge through shared memory; the sink enters
@@ -591,6 +592,275 @@ chunk_attention_group_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
             }
         }
     }
+}
+
+// ------------------------------------------------------------------------------------------------- head-tile decode kernel
+// The same rows for head sizes the tensor cores take (dk a multiple of 32, dv one of the prompt kernel's sizes): one CTA per
+// (row, kv head), the query heads of that kv head as the rows of a 16-row operand (two maps: rows 0 - 7 hold the first maps of
+// eight heads, rows 8 - 15 their second), so a K or V row is read once and multiplied for all of them at once.  Four warps take
+// 32 visible keys at a time each, gather their K and V rows from the pages with cp.async (four lanes a row, one page lookup per
+// key), run S = Q K^T and O += P V on mma.sync with the softmax in the accumulator registers, and merge through shared
+// memory, which by then no longer holds tiles.  The keys a single row sees are one exact range: nothing to mask but its end.
+constexpr int kHeadRows = 16, kHeadKeys = 32;
+
+template <int DVT, bool SIG, int MAPS>
+__global__ void __launch_bounds__(128)
+chunk_attention_heads_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
+                             const __nv_bfloat16* __restrict__ v_cache, const int32_t* __restrict__ block_tables, int max_nb,
+                             const int32_t* __restrict__ cu_q, const int32_t* __restrict__ ctx_start, int n_seq, int H, int G,
+                             int dk, int bs, float scale_log2, int chunk, int window, int keep_first, float sink,
+                             float sink_logit, const float* __restrict__ sink_logits, const float* __restrict__ head_bias,
+                             const __nv_bfloat16* __restrict__ gate, int64_t gate_stride, HeadShape hs, int skip_rows_from,
+                             __nv_bfloat16* __restrict__ out, int64_t out_stride) {
+    constexpr int DV = 16 * DVT, LDV = DV + 8, PASS = kHeadRows / MAPS, PW = 2 + DV;
+    constexpr float kLog2e = 1.4426950408889634f;
+    // q [16][dk + 8], then per warp: K tile [32][MAPS * dk + 8], V tile [32][DV + 8]; the merge reuses the tiles' place
+    extern __shared__ __align__(16) unsigned char head_sm[];
+    const int row = blockIdx.x, g = blockIdx.y;
+    const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+    const int seq = b2::seq_of_row(cu_q, n_seq, row);
+    const int ctx = ctx_start[seq];
+    const int QHall = H / G;
+    if (skip_rows_from > 0 && ctx >= 0 && cu_q[seq + 1] - cu_q[seq] >= skip_rows_from) return;    // the tile kernel's
+    if (ctx < 0) {
+        for (int i = tid; i < QHall * DV; i += 128)
+            out[(size_t)row * out_stride + (size_t)g * QHall * DV + i] = __float2bfloat16_rn(0.f);
+        return;
+    }
+    const int pos = ctx + row - cu_q[seq];
+    const KeySpan span = key_span(pos, pos, chunk, window, keep_first);
+    const int32_t* bt = block_tables + (size_t)seq * max_nb;
+    const int ldq = dk + 8, ldk = MAPS * dk + 8;
+    __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(head_sm);
+    __nv_bfloat16* tiles = q_sm + kHeadRows * ldq;
+    __nv_bfloat16* kt = tiles + (size_t)w * kHeadKeys * (ldk + LDV);
+    __nv_bfloat16* vt = kt + kHeadKeys * ldk;
+    float* part = reinterpret_cast<float*>(tiles);       // [4][16][m, l, O (DV)]
+    const uint32_t q_base = b2::smem_u32(q_sm), k_base = b2::smem_u32(kt), v_base = b2::smem_u32(vt);
+    const int gq = lane >> 2, tq = lane & 3;
+    const float cap_log2 = hs.cap * kLog2e, cap_e = hs.cap > 0.f ? 2.f / hs.cap : 0.f;
+
+    for (int h0 = 0; h0 < QHall; h0 += PASS) {
+        const int QH = min(PASS, QHall - h0);
+        __syncthreads();                                 // a previous pass is done with the shared memory
+        for (int idx = tid; idx < kHeadRows * (dk / 8); idx += 128) {
+            const int r = idx / (dk / 8), c = (idx % (dk / 8)) * 8, h = r % PASS, mp = r / PASS;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (h < QH) v = *reinterpret_cast<const uint4*>(q + (((size_t)row * H + (size_t)g * QHall + h0 + h) * MAPS + mp) * dk + c);
+            *reinterpret_cast<uint4*>(q_sm + r * ldq + c) = v;
+        }
+        __syncthreads();
+        // this thread's two rows and the heads they belong to
+        const int ha = g * QHall + h0 + min(gq, QH - 1), hb = MAPS > 1 ? ha : g * QHall + h0 + min(gq + 8, QH - 1);
+        float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, ba = 0.f, bb = 0.f;
+        if (w == 0 && sink > 0.f) {                      // the sink enters once, through the first warp
+            m0 = (sink_logits ? sink_logits[ha] : sink_logit) * kLog2e;
+            m1 = (sink_logits ? sink_logits[hb] : sink_logit) * kLog2e;
+            l0 = l1 = tq == 0 ? sink : 0.f;
+        }
+        if (SIG && head_bias) {
+            ba = head_bias[ha] * kLog2e;
+            bb = head_bias[hb] * kLog2e;
+        }
+        float o[2 * DVT][4];
+#pragma unroll
+        for (int n = 0; n < 2 * DVT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+
+        for (int c0 = w * kHeadKeys; c0 < span.n; c0 += 4 * kHeadKeys) {
+            // keys past the end repeat the last one: finite numbers that the mask drops
+            const int j = span.key(min(c0 + lane, span.n - 1));
+            const int page = bt[j / bs], off = j % bs;
+            __syncwarp();                                // the previous tile has been read
+#pragma unroll
+            for (int kq = 0; kq < kHeadKeys / 8; ++kq) {
+                const int key = kq * 8 + (lane >> 2), c = (lane & 3) * 8;
+                const size_t pg = __shfl_sync(0xffffffffu, page, key);
+                const int of = __shfl_sync(0xffffffffu, off, key);
+#pragma unroll
+                for (int mp = 0; mp < MAPS; ++mp) {
+                    const __nv_bfloat16* ks = k_cache + ((pg * (G * MAPS) + g * MAPS + mp) * bs + of) * dk + c;
+                    __nv_bfloat16* kd = kt + key * ldk + mp * dk + c;
+                    for (int t = 0; t < dk; t += 32) cp_async16(kd + t, ks + t);
+                }
+                const __nv_bfloat16* vs = v_cache + ((pg * G + g) * bs + of) * DV + c;
+                __nv_bfloat16* vd = vt + key * LDV + c;
+#pragma unroll
+                for (int t = 0; t < DV; t += 32) cp_async16(vd + t, vs + t);
+            }
+            asm volatile("cp.async.commit_group;" ::: "memory");
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+            __syncwarp();
+            float sc[4][4], sd[MAPS > 1 ? 4 : 1][4];
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+                sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+                if (MAPS > 1) sd[MAPS > 1 ? n : 0][0] = sd[MAPS > 1 ? n : 0][1] = sd[MAPS > 1 ? n : 0][2] = sd[MAPS > 1 ? n : 0][3] = 0.f;
+            }
+            for (int kk = 0; kk < dk; kk += 16) {
+                uint32_t a0, a1, a2, a3;
+                b2::ldmatrix_x4(q_base + 2u * ((lane & 15) * ldq + kk + (lane >> 4) * 8), a0, a1, a2, a3);
+#pragma unroll
+                for (int n2 = 0; n2 < 2; ++n2) {
+                    uint32_t b0, b1, b2_, b3;
+                    const int key = n2 * 16 + (lane >> 4) * 8 + (lane & 7), dim = kk + ((lane >> 3) & 1) * 8;
+                    b2::ldmatrix_x4(k_base + 2u * (key * ldk + dim), b0, b1, b2_, b3);
+                    b2::mma_bf16_16816(sc[2 * n2], a0, a1, a2, a3, b0, b1);
+                    b2::mma_bf16_16816(sc[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
+                    if (MAPS > 1) {                      // rows 8 - 15 belong to the second maps and take their keys
+                        b2::ldmatrix_x4(k_base + 2u * (key * ldk + dk + dim), b0, b1, b2_, b3);
+                        b2::mma_bf16_16816(sd[MAPS > 1 ? 2 * n2 : 0], a0, a1, a2, a3, b0, b1);
+                        b2::mma_bf16_16816(sd[MAPS > 1 ? 2 * n2 + 1 : 0], a0, a1, a2, a3, b2_, b3);
+                    }
+                }
+            }
+            if (MAPS > 1) {
+#pragma unroll
+                for (int n = 0; n < 4; ++n) {
+                    sc[n][2] = sd[MAPS > 1 ? n : 0][2];
+                    sc[n][3] = sd[MAPS > 1 ? n : 0][3];
+                }
+            }
+            const bool whole = c0 + kHeadKeys <= span.n;
+            float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    float x = sc[n][e] * scale_log2;
+                    const bool in = whole || c0 + n * 8 + 2 * tq + (e & 1) < span.n;
+                    if (SIG) {
+                        x = in ? sigmoid2_f(x + (e < 2 ? ba : bb)) : 0.f;
+                    } else {
+                        if (hs.cap > 0.f) x = cap_score(x, cap_log2, cap_e);
+                        if (!in) x = -INFINITY;
+                        if (e < 2) mx0 = fmaxf(mx0, x); else mx1 = fmaxf(mx1, x);
+                    }
+                    sc[n][e] = x;
+                }
+            }
+            if (!SIG) {
+#pragma unroll
+                for (int x = 1; x < 4; x <<= 1) {
+                    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, x));
+                    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, x));
+                }
+                const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);         // finite: the tile has at least one key
+                const float f0 = b2::fast_exp2(m0 - mn0), f1 = b2::fast_exp2(m1 - mn1);
+                m0 = mn0;
+                m1 = mn1;
+                l0 *= f0;
+                l1 *= f1;
+#pragma unroll
+                for (int n = 0; n < 4; ++n) {
+                    sc[n][0] = b2::fast_exp2(sc[n][0] - mn0);
+                    sc[n][1] = b2::fast_exp2(sc[n][1] - mn0);
+                    sc[n][2] = b2::fast_exp2(sc[n][2] - mn1);
+                    sc[n][3] = b2::fast_exp2(sc[n][3] - mn1);
+                    l0 += sc[n][0] + sc[n][1];
+                    l1 += sc[n][2] + sc[n][3];
+                }
+#pragma unroll
+                for (int n = 0; n < 2 * DVT; ++n) {
+                    o[n][0] *= f0;
+                    o[n][1] *= f0;
+                    o[n][2] *= f1;
+                    o[n][3] *= f1;
+                }
+            }
+#pragma unroll
+            for (int ks = 0; ks < 2; ++ks) {
+                const uint32_t a0 = b2::pack_bf16x2(sc[2 * ks][0], sc[2 * ks][1]), a1 = b2::pack_bf16x2(sc[2 * ks][2], sc[2 * ks][3]);
+                const uint32_t a2 = b2::pack_bf16x2(sc[2 * ks + 1][0], sc[2 * ks + 1][1]),
+                               a3 = b2::pack_bf16x2(sc[2 * ks + 1][2], sc[2 * ks + 1][3]);
+#pragma unroll
+                for (int n2 = 0; n2 < DVT; ++n2) {
+                    uint32_t b0, b1, b2_, b3;
+                    const int key = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), col = n2 * 16 + (lane >> 4) * 8;
+                    b2::ldmatrix_x4_trans(v_base + 2u * (key * LDV + col), b0, b1, b2_, b3);
+                    b2::mma_bf16_16816(o[2 * n2], a0, a1, a2, a3, b0, b1);
+                    b2::mma_bf16_16816(o[2 * n2 + 1], a0, a1, a2, a3, b2_, b3);
+                }
+            }
+        }
+#pragma unroll
+        for (int x = 1; x < 4; x <<= 1) {
+            l0 += __shfl_xor_sync(0xffffffffu, l0, x);
+            l1 += __shfl_xor_sync(0xffffffffu, l1, x);
+        }
+        __syncthreads();                                 // every warp is done with its tiles: the partial results take their place
+        float* pa = part + (size_t)(w * kHeadRows + gq) * PW;
+        float* pb = pa + 8 * PW;
+        if (tq == 0) {
+            pa[0] = m0; pa[1] = l0;
+            pb[0] = m1; pb[1] = l1;
+        }
+#pragma unroll
+        for (int n = 0; n < 2 * DVT; ++n) {
+            const int col = 2 + n * 8 + 2 * tq;
+            *reinterpret_cast<float2*>(pa + col) = make_float2(o[n][0], o[n][1]);
+            *reinterpret_cast<float2*>(pb + col) = make_float2(o[n][2], o[n][3]);
+        }
+        __syncthreads();
+        // a warp per head: merged output of operand row r at column col
+        for (int h = w; h < QH; h += 4) {
+            const size_t head = (size_t)g * QHall + h0 + h;
+            float f[MAPS][4];
+#pragma unroll
+            for (int mp = 0; mp < MAPS; ++mp) {
+                const float* px = part + (size_t)(h + mp * PASS) * PW;
+                float M = -INFINITY, L = 0.f;
+#pragma unroll
+                for (int x = 0; x < 4; ++x) M = fmaxf(M, px[(size_t)x * kHeadRows * PW]);
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                    const float mx = px[(size_t)x * kHeadRows * PW];
+                    f[mp][x] = SIG ? 1.f : (mx == -INFINITY ? 0.f : b2::fast_exp2(mx - M));
+                    L = fmaf(px[(size_t)x * kHeadRows * PW + 1], f[mp][x], L);
+                }
+                const float inv = (SIG ? 1.f : (L > 0.f ? 1.f / L : 0.f)) * (mp == 0 ? 1.f : -hs.lambda);
+#pragma unroll
+                for (int x = 0; x < 4; ++x) f[mp][x] *= inv;
+            }
+            float v[DV / 32], ss = 0.f;
+#pragma unroll
+            for (int c = 0; c < DV / 32; ++c) {
+                v[c] = 0.f;
+#pragma unroll
+                for (int mp = 0; mp < MAPS; ++mp) {
+                    const float* px = part + (size_t)(h + mp * PASS) * PW + 2 + lane + 32 * c;
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) v[c] = fmaf(px[(size_t)x * kHeadRows * PW], f[mp][x], v[c]);
+                }
+                ss = fmaf(v[c], v[c], ss);
+            }
+            float inv = MAPS > 1 ? rsqrtf(b2::warp_sum(ss) / (float)DV + hs.eps) * hs.out_scale : 1.f;
+            if (gate) inv *= b2::sigmoid_f(__bfloat162float(gate[(size_t)row * gate_stride + head]));
+#pragma unroll
+            for (int c = 0; c < DV / 32; ++c)
+                out[(size_t)row * out_stride + head * DV + lane + 32 * c] = __float2bfloat16_rn(v[c] * inv);
+        }
+    }
+}
+
+template <int DVT, bool SIG, int MAPS>
+int launch_heads(const void* q, const void* k_cache, const void* v_cache, const int32_t* block_tables, int max_nb,
+                 const int32_t* cu_q, const int32_t* ctx_start, int n_seq, int T, int H, int G, int dk, int bs, float scale, int chunk,
+                 int window, int keep_first, float sink, float sink_logit, const float* sink_logits, const float* head_bias,
+                 const void* gate, int64_t gate_stride, const HeadShape& hs, int skip_from, void* out, int64_t out_stride,
+                 cudaStream_t st) {
+    constexpr int DV = 16 * DVT;
+    const size_t tiles = (size_t)4 * kHeadKeys * (MAPS * dk + 8 + DV + 8) * sizeof(__nv_bfloat16);
+    const size_t merge = (size_t)4 * kHeadRows * (2 + DV) * sizeof(float);
+    const size_t smem = (size_t)kHeadRows * (dk + 8) * sizeof(__nv_bfloat16) + (tiles > merge ? tiles : merge);
+    auto kern = chunk_attention_heads_kernel<DVT, SIG, MAPS>;
+    if (smem > 48 * 1024) B2_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    kern<<<dim3(T, G), 128, smem, st>>>(static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
+                                       static_cast<const __nv_bfloat16*>(v_cache), block_tables, max_nb, cu_q, ctx_start, n_seq, H,
+                                       G, dk, bs, scale * 1.4426950408889634f, chunk, window, keep_first, sink, sink_logit, sink_logits,
+                                       head_bias, static_cast<const __nv_bfloat16*>(gate), gate_stride, hs, skip_from,
+                                       static_cast<__nv_bfloat16*>(out), out_stride);
+    B2_CUDA_OK(cudaGetLastError());
+    return B2_OK;
 }
 
 // ------------------------------------------------------------------------------------------------- tiled prompt kernel
@@ -1038,6 +1308,18 @@ extern "C" int b2_masked_attention(void* out, const void* q, const void* k_cache
 #undef B2_TILE_WIDE
 #undef B2_TILE_RUN
         if (rc != B2_OK) return rc;
+    }
+    if (act_dtype == B2_ACT_BF16 && dk % 32 == 0 && dk <= 256 && b2_aligned16(q) && b2_aligned16(k_cache) && b2_aligned16(v_cache)) {
+        int rc = B2_EUNSUPPORTED;
+#define B2_HEADS_RUN(b, SIG, MAPS)                                                                                        \
+    launch_heads<b, SIG, MAPS>(q, k_cache, v_cache, block_tables, max_nb, cu_q, ctx_start, n_seq, T, H, G, dk, bs, scale, chunk, \
+                               window, keep_first, sink, sink_logit, sink_logits, head_bias, gate, gate_stride, hs, skip_from, out, \
+                               out_stride, st)
+#define B2_HEADS(b) if (dv == 16 * b) rc = sig ? B2_HEADS_RUN(b, true, 1) : (maps == 2 ? B2_HEADS_RUN(b, false, 2) : B2_HEADS_RUN(b, false, 1));
+        B2_HEADS(2) B2_HEADS(4) B2_HEADS(6) B2_HEADS(8) B2_HEADS(12) B2_HEADS(16)
+#undef B2_HEADS
+#undef B2_HEADS_RUN
+        if (rc != B2_EUNSUPPORTED) return rc;
     }
     if (act_dtype == B2_ACT_BF16 && dk % 8 == 0 && dv % 8 == 0 && dv <= 64 * kGroupMaxPairs && b2_aligned16(q) &&
         b2_aligned16(k_cache) && b2_aligned16(v_cache) && b2_aligned16(out)) {

@@ -147,6 +147,111 @@ sandwich_norm_kernel(float* __restrict__ x, int D, const T* __restrict__ y, int6
     }
 }
 
+// RMS norms without biases on rows of up to 8192: the residual and the sublayer's rows are loaded at once and stay in registers
+// (N accesses of four a thread), so the op waits for memory once and every reduction costs one barrier.
+constexpr int kRmsThreads = 512;
+
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {        // red: one slot per warp, used once
+    a = b2::warp_sum(a);
+    b = b2::warp_sum(b);
+    const int nw = (blockDim.x + 31) >> 5;
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+    __syncthreads();
+    a = b = 0.f;
+    for (int x = 0; x < nw; ++x) {
+        a += red[x].x;
+        b += red[x].y;
+    }
+    return make_float2(a, b);
+}
+
+template <typename T, int N, bool PAIR>
+__global__ void __launch_bounds__(kRmsThreads)
+sandwich_rms_kernel(float* __restrict__ x, int D, const T* __restrict__ y, int64_t y_stride, PairRows<T> pair, const float* __restrict__ post_w,
+                    const float* __restrict__ pre_w, float eps, T* __restrict__ h, int64_t h_stride) {
+    __shared__ float2 red[3][kRmsThreads / 32];
+    const int t = blockIdx.x, step = blockDim.x * 4;
+    float* xt = x + (size_t)t * D;
+    float r[N][4], a[N][4], b[PAIR ? N : 1][4];
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int d = threadIdx.x * 4 + n * step;
+        r[n][0] = r[n][1] = r[n][2] = r[n][3] = 0.f;
+        a[n][0] = a[n][1] = a[n][2] = a[n][3] = 0.f;
+        if (PAIR) b[PAIR ? n : 0][0] = b[PAIR ? n : 0][1] = b[PAIR ? n : 0][2] = b[PAIR ? n : 0][3] = 0.f;
+        if (d < D) {
+            b2::ld4(xt + d, r[n]);
+            if (y) b2::ld4(y + (size_t)t * y_stride + d, a[n]);
+            if (PAIR) b2::ld4(pair.y2 + (size_t)t * pair.y2_stride + d, b[PAIR ? n : 0]);
+        }
+    }
+    if (y) {
+        if (PAIR) {
+            float s1 = 0.f, s2 = 0.f;
+#pragma unroll
+            for (int n = 0; n < N; ++n) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    s1 = fmaf(a[n][c], a[n][c], s1);
+                    s2 = fmaf(b[PAIR ? n : 0][c], b[PAIR ? n : 0][c], s2);
+                }
+            }
+            const float2 ss = block_sum2(s1, s2, red[0]);
+            const float i1 = rsqrtf(ss.x / (float)D + eps) * pair.scale, i2 = rsqrtf(ss.y / (float)D + eps) * pair.scale;
+#pragma unroll
+            for (int n = 0; n < N; ++n) {
+                const int d = threadIdx.x * 4 + n * step;
+                if (d < D) {
+                    const float4 u = *reinterpret_cast<const float4*>(pair.w1 + d), v = *reinterpret_cast<const float4*>(pair.w2 + d);
+                    const float wu[4] = {u.x, u.y, u.z, u.w}, wv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) a[n][c] = a[n][c] * i1 * wu[c] + b[PAIR ? n : 0][c] * i2 * wv[c];
+                }
+            }
+        }
+        float inv = 1.f;
+        if (post_w) {
+            float s1 = 0.f;
+#pragma unroll
+            for (int n = 0; n < N; ++n) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c) s1 = fmaf(a[n][c], a[n][c], s1);
+            }
+            inv = rsqrtf(block_sum2(s1, 0.f, red[1]).x / (float)D + eps);
+        }
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            const int d = threadIdx.x * 4 + n * step;
+            if (d < D) {
+                float wp[4] = {1.f, 1.f, 1.f, 1.f};
+                if (post_w) b2::ld4(post_w + d, wp);
+#pragma unroll
+                for (int c = 0; c < 4; ++c) r[n][c] += a[n][c] * inv * wp[c];
+                b2::st4(xt + d, r[n]);
+            }
+        }
+    }
+    if (!h) return;
+    float s1 = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) s1 = fmaf(r[n][c], r[n][c], s1);
+    }
+    const float inv = rsqrtf(block_sum2(s1, 0.f, red[2]).x / (float)D + eps);
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int d = threadIdx.x * 4 + n * step;
+        if (d < D) {
+            float wn[4];
+            b2::ld4(pre_w + d, wn);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) wn[c] *= r[n][c] * inv;
+            b2::st4(h + (size_t)t * h_stride + d, wn);
+        }
+    }
+}
+
 // W = 4: 16-byte (fp32) or 8-byte (bf16) accesses, the row kept in registers between the two passes when it fits (up to
 // kRowNormKeep accesses a thread); W = 1: any width and alignment.
 constexpr int kRowNormKeep = 4;
@@ -330,6 +435,25 @@ static int sandwich_norm(float* x, int T, int D, const void* y, int64_t y_stride
     const int threads = D >= 8192 ? 512 : (D >= 1024 ? 256 : 128);
     const bool vec = D % 4 == 0 && (!y || (y_stride % 4 == 0 && b2_aligned16(y))) && (!h || (h_stride % 4 == 0 && b2_aligned16(h))) &&
                      (!y2 || (y2_stride % 4 == 0 && b2_aligned16(y2)));
+    if (vec && norm_kind == B2_NORM_RMS && !post_b && !pre_b && D <= 16 * kRmsThreads && (!post_w || b2_aligned16(post_w)) &&
+        (!h || b2_aligned16(pre_w)) && (!y2 || (b2_aligned16(w1) && b2_aligned16(w2)))) {
+        const int per = D <= 1024 ? 1 : (D <= 8 * kRmsThreads ? 2 : 4);
+        const int nt = ((D + 4 * per - 1) / (4 * per) + 31) / 32 * 32;
+#define B2_RMS(N, PAIR)                                                                                                     \
+    sandwich_rms_kernel<A, N, PAIR><<<T, nt, 0, st>>>(x, D, static_cast<const A*>(y), y_stride,                             \
+                                                      PairRows<A>{static_cast<const A*>(y2), y2_stride, w1, w2, pair_scale}, post_w, \
+                                                      pre_w, eps, static_cast<A*>(h), h_stride)
+        B2_DISPATCH_ACT(act_dtype, A, {
+            if (y2) {
+                if (per == 1) B2_RMS(1, true); else if (per == 2) B2_RMS(2, true); else B2_RMS(4, true);
+            } else {
+                if (per == 1) B2_RMS(1, false); else if (per == 2) B2_RMS(2, false); else B2_RMS(4, false);
+            }
+        });
+#undef B2_RMS
+        B2_CUDA_OK(cudaGetLastError());
+        return B2_OK;
+    }
 #define B2_SANDWICH(W, PAIR)                                                                                                \
     do {                                                                                                                    \
         auto kern = sandwich_norm_kernel<A, W, PAIR>;                                                                       \
