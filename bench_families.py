@@ -1,10 +1,12 @@
-"""`bench.py --family kofadra|gatolix|tonilix|sanarax|gapidra`: prefill and decode throughput of a model family at layer sizes of real models
+"""`bench.py --family kofadra|gatolix|tonilix|sanarax|gapidra|lizazen`: prefill and decode throughput of a model family at layer sizes of real models
 (random weights), beside the Llama model of equal width, heads, head size and ACTIVE feed-forward width, plus the device
 time of every kernel of the family with the roofline that bounds it beside the like kernel of the Llama path (Tonilix:
 beside the Kofadra family, whose recurrent mixer, attention without rotation and routed experts are the closest; Sanarax:
 beside the Gatolix family, whose norms on both sides, latent attention and squared-ReLU feed-forward are the closest, with
 the like kernel of Kofadra and Tonilix for the sink attention and the linear attention; Gapidra: beside Sanarax, whose
-windowed grouped-query attention, latent attention and dense ungated feed-forward are the closest).
+windowed grouped-query attention, latent attention and dense ungated feed-forward are the closest; Lizazen: beside Tonilix, whose
+parallel mixer of attention and linear attention and routed experts are the closest, with the like kernels of Sanarax, Gapidra and
+Kofadra for the norms and the attention).
 
 Both models run through the same engine (LLMEngine.replay_step: scheduler, pools, state slots, CUDA-graph decode).
   prefill   one prompt chunk of T tokens in one step; wall clock around the step (it ends with a stream synchronize)
@@ -48,6 +50,10 @@ SANARAX_SIZES = {
 
 # Gapidra: the same widths, heads and latent; latent and sigmoid-attention layers in turn (no query latent)
 GAPIDRA_SIZES = {k: dict({n: v for n, v in s.items() if n not in ("q_rank", "keep_first")}, layers=6) for k, s in SANARAX_SIZES.items()}
+
+
+# Lizazen: the head geometry, experts and widths of SIZES; six layers = two of each mixer
+LIZAZEN_SIZES = {k: dict(s, layers=6, window=1024, keep_first=4, chunk=1024) for k, s in SIZES.items()}
 
 
 def _peaks():
@@ -744,10 +750,150 @@ def _kernels_gapidra(size, s, B, ctx, T):
         torch.cuda.empty_cache()
 
 
+def _kernels_lizazen(size, s, B, ctx, T):
+    """Device time of the kernels of a Lizazen layer, each beside the like kernel of an existing family on the same shapes."""
+    import torch
+    from b200attn import ops
+    dev = torch.device("cuda", 0)
+    HBM, TF, src = _peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    D, H, G, d, F, E, top, W, keep, Ck = (s[k] for k in ("hidden", "heads", "kv_heads", "head_dim", "ff", "experts", "top", "window",
+                                                         "keep_first", "chunk"))
+    bf = torch.bfloat16
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)          # noqa: E731
+    rand = lambda *sh: torch.randn(*sh, device=dev).to(bf)          # noqa: E731
+
+    def line(kernel, phase, ms, bytes_=0, flops=0, like=None):
+        gbs, tfs = bytes_ / ms / 1e6, flops / ms / 1e9
+        _emit(bench="kernel", size=size, kernel=kernel, phase=phase, ms=round(ms, 4), gb_per_s=round(gbs, 1),
+              tflop_per_s=round(tfs, 2), frac_hbm=round(gbs / HBM, 3), frac_bf16=round(tfs / TF, 4), peaks=src, like=like)
+
+    zones = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}
+    tab_w = ops.rotary_table(ctx + T + 64, d, 5e5, zones, dev)
+    tab_h = ops.rotary_table(ctx + T + 64, d // 2, 1e6, None, dev)
+    tab_r = ops.rotary_table(ctx + T + 64, d, 1e4, None, dev)
+    for phase, n_seq, q_len, c in (("prefill", 1, T, 0), ("decode", B, 1, ctx)):
+        rows = n_seq * q_len
+        nb_seq = (c + q_len + 15) // 16
+        tables = torch.arange(n_seq * nb_seq, dtype=torch.int32, device=dev).view(n_seq, nb_seq)
+        batch = ops.SeqBatch(i32([i * q_len for i in range(n_seq + 1)]), i32([c] * n_seq), tables, i32(list(range(n_seq))), n_seq, rows)
+        pos = (torch.arange(rows, device=dev) % q_len + c).to(torch.int32)
+        slots = (torch.arange(rows, device=dev) // q_len * (nb_seq * 16) + pos).to(torch.int64)
+        one = torch.ones(D, device=dev)
+        # ---- embedding + hashed bigram row  |  like: the plain embedding
+        emb, big = rand(s["vocab"], D), rand(65522, D)
+        tok = torch.randint(0, s["vocab"], (rows,), device=dev)
+        last = torch.zeros(n_seq, dtype=torch.int64, device=dev)
+        ms = _time(lambda: ops.embed_bigram(emb, big, tok, batch, 1009, 31, last), flush)
+        line("embed_bigram", phase, ms, bytes_=rows * D * (2 + 2 + 4), like="embed_streams (Kofadra)")
+        ms = _time(lambda: ops.embed_streams(emb, tok, 1, 1.0), flush)
+        line("embed_streams (Kofadra, 1 stream)", phase, ms, bytes_=rows * D * (2 + 4))
+        del emb, big
+        # ---- the two halves' norms, their sum, the norm after it, the residual, the next norm  |  like: norms on both sides
+        x, y, y2 = torch.randn(rows, D, device=dev), rand(rows, D), rand(rows, D)
+        ms = _time(lambda: ops.sandwich_norm_pair(x, y, one, y2, one, 0.5, one, one, 1e-6), flush)
+        line("sandwich_norm_pair (4 RMS norms, two halves)", phase, ms, bytes_=rows * D * 14, like="sandwich_norm (Sanarax)")
+        ms = _time(lambda: ops.sandwich_norm(x, y, one, None, one, None, eps=1e-6, norm_kind=ops.NORM_RMS), flush)
+        line("sandwich_norm (Sanarax, 2 RMS norms)", phase, ms, bytes_=rows * D * 12)
+        # ---- capped attention on its own keys: norms + rotation + pool write  |  like: Gapidra's
+        kc, vc = rand(n_seq * nb_seq, G, 16, d), rand(n_seq * nb_seq, G, 16, d)
+        qkv = rand(rows, (H + 2 * G) * d)
+        nq, nk = torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+        ms = _time(lambda: ops.qk_rope_cache(qkv, H, G, d, d, pos, tab_w, d, slots, kc, vc, v_from_k=True, q_norm=nq, k_norm=nk), flush)
+        line("qk_norm_rope_cache (values = keys as projected)", phase, ms, bytes_=rows * (2 * H + 3 * G) * d * 2, like="qk_norm_rope_cache (Gapidra)")
+        ms = _time(lambda: ops.qk_rope_cache(qkv, H, G, d, d, pos, tab_h, d // 2, slots, kc, vc, interleaved=True, q_norm=nq, k_norm=nk), flush)
+        line("qk_norm_rope_cache (Gapidra)", phase, ms, bytes_=rows * (2 * H + 4 * G) * d * 2)
+        q, sinks, hg = rand(rows, H, d), torch.randn(H, device=dev), rand(rows, H)
+        pairs = sum(min(p + 1, W) for p in range(T))
+        kept = sum(min(p + 1, W) + max(0, min(keep, p - W + 1)) for p in range(T))
+        seen = min(c + 1, W)
+        per_key = n_seq * G * 2 * d * 2
+        work = (lambda n, f: dict(flops=f * n * H)) if phase == "prefill" else (lambda n, f: dict(bytes_=per_key * n))
+        ms = _time(lambda: ops.chunk_attention(q, kc, vc, batch, d ** -0.5, window=W, sink=1.0, sink_logits=sinks, softcap=50.0), flush)
+        line("chunk_attention (window %d, capped scores, sink)" % W, phase, ms, like="chunk_attention (Sanarax)",
+             **work(pairs if phase == "prefill" else seen, 4 * d))
+        ms = _time(lambda: ops.chunk_attention(q, kc, vc, batch, d ** -0.5, window=W, sink=1.0, sink_logits=sinks, gate=hg), flush)
+        line("chunk_attention (Sanarax: window %d, sink, gate)" % W, phase, ms, **work(pairs if phase == "prefill" else seen, 4 * d))
+        # ---- differential attention: two maps of half the head size over values of d
+        kd = kc.view(n_seq * nb_seq, 2 * G, 16, d // 2)
+        ms = _time(lambda: ops.qk_rope_cache(qkv, 2 * H, 2 * G, d // 2, d, pos, tab_h, d // 2, slots, kd, vc), flush)
+        line("qk_rope_cache (two maps per head)", phase, ms, bytes_=rows * (2 * H + 4 * G) * d * 2, like="qk_rope_cache (Sanarax)")
+        ms = _time(lambda: ops.qk_rope_cache(qkv, H, G, d, d, pos, tab_h, d // 2, slots, kc, vc), flush)
+        line("qk_rope_cache (Sanarax, half of every head turns)", phase, ms, bytes_=rows * (2 * H + 4 * G) * d * 2)
+        qd = q.view(rows, 2 * H, d // 2)
+        ms = _time(lambda: ops.chunk_attention(qd, kd, vc, batch, (d // 2) ** -0.5, window=W, keep_first=keep, maps=2, map_lambda=0.4,
+                                               map_scale=0.6), flush)
+        nk_ = kept if phase == "prefill" else seen + keep
+        line("chunk_attention (differential, window %d + %d kept)" % (W, keep), phase, ms, like="chunk_attention (Sanarax, kept)", **work(nk_, 6 * d))
+        ms = _time(lambda: ops.chunk_attention(q, kc, vc, batch, d ** -0.5, window=W, keep_first=keep, sink=1.0, sink_logits=sinks, gate=hg), flush)
+        line("chunk_attention (Sanarax, window %d + %d kept)" % (W, keep), phase, ms, **work(nk_, 4 * d))
+        # ---- chunked attention, values of the key size and twice that  |  like: Kofadra's blocks
+        cp = sum(p % Ck + 1 for p in range(T)) if phase == "prefill" else c % Ck + 1
+        ms = _time(lambda: ops.chunk_attention(q, kc, vc, batch, d ** -0.5, Ck), flush)
+        line("chunk_attention (blocks of %d)" % Ck, phase, ms, like="chunk_attention (Kofadra)", **work(cp, 4 * d))
+        ms = _time(lambda: ops.chunk_attention(q, kc, vc, batch, d ** -0.5, Ck, sink=1.0), flush)
+        line("chunk_attention (Kofadra: blocks of %d, sink)" % Ck, phase, ms, **work(cp, 4 * d))
+        vw = rand(n_seq * nb_seq, G, 16, 2 * d)
+        ms = _time(lambda: ops.chunk_attention(q, kc, vw, batch, d ** -0.5, Ck), flush)
+        ww = work(cp, 6 * d) if phase == "prefill" else dict(bytes_=per_key * cp * 3 // 2)
+        line("chunk_attention (blocks of %d, values of %d)" % (Ck, 2 * d), phase, ms, like="chunk_attention (Kofadra)", **ww)
+        del kc, vc, vw, kd, qkv, q, qd
+        # ---- retention  |  like: Sanarax's and Tonilix's linear attention
+        R = max(H // 2, 1)
+        C = 3 * R * d
+        lp = rand(rows, C + R * d)
+        dec = torch.full((R,), 0.99, device=dev)
+        prep = lambda **k: ops.recur_prep(lp, R, R, d, d, batch, decay_mode=ops.DECAY_HEAD_CONST, decay_bias=dec, **k)          # noqa: E731
+        ms = _time(lambda: prep(k_scale=d ** -0.5, cos_sin=tab_r), flush)
+        line("recur_prep (rotated q and k, fixed decay)", phase, ms, bytes_=rows * (C * 2 + C * 4 + 4 * R), like="recur_prep (Sanarax)")
+        ms = _time(lambda: prep(conv_silu=True), flush)
+        line("recur_prep (Sanarax: SiLU, fixed decay)", phase, ms, bytes_=rows * (C * 2 + C * 4 + 4 * R))
+        state = torch.zeros(n_seq, R, d, d, device=dev)
+        q32, _, decay = prep(k_scale=d ** -0.5, cos_sin=tab_r)
+        io = n_seq * R * d * d * 4 * 2 + rows * (C + R * d) * 4
+        ms = _time(lambda: ops.channel_scan(q32, None, decay, R, R, d, d, batch, state, delta=False), flush)
+        line("channel_scan (fixed decay per head)", phase, ms, flops=6 * rows * R * d * d, bytes_=io, like="channel_scan (Tonilix)")
+        dch = torch.rand(rows, R * d, device=dev)
+        ms = _time(lambda: ops.channel_scan(q32, None, dch, R, R, d, d, batch, state, delta=False), flush)
+        line("channel_scan (Tonilix: decay per key channel)", phase, ms, flops=6 * rows * R * d * d, bytes_=io + rows * R * d * 4)
+        o32 = torch.randn(rows, R, d, device=dev)
+        ms = _time(lambda: ops.gated_head_norm(o32, lp[:, C:], None, 1e-6, ops.GATE_SILU), flush)
+        line("gated_head_norm (no weight)", phase, ms, bytes_=rows * R * d * 8, like="gated_head_norm (Tonilix)")
+        nd = torch.ones(d, device=dev)
+        ms = _time(lambda: ops.gated_head_norm(o32, lp[:, C:], nd, 1e-6, ops.GATE_SILU), flush)
+        line("gated_head_norm (Tonilix)", phase, ms, bytes_=rows * R * d * 8)
+        del lp, q32, dch, state, o32
+        # ---- feed-forwards  |  like: Kofadra's and Tonilix's router and experts, the Llama gated unit
+        gu = rand(rows, 2 * top * F)
+        ms = _time(lambda: ops.glu_and_mul(gu, ops.GLU_CLAMPED, 1.702, 7.0), flush)
+        line("glu_and_mul (bounded units)", phase, ms, bytes_=rows * top * F * 6, like="silu_and_mul (Llama)")
+        ms = _time(lambda: ops.glu_and_mul(gu, ops.GLU_SILU), flush)
+        line("glu_and_mul (SiLU, the shared expert's)", phase, ms, bytes_=rows * top * F * 6, like="silu_and_mul (Llama)")
+        ms = _time(lambda: ops.silu_and_mul(gu), flush)
+        line("silu_and_mul (Llama)", phase, ms, bytes_=rows * top * F * 6)
+        h, wr, rb = rand(rows, D), (torch.randn(E, D, device=dev) * D ** -0.5).to(bf), torch.zeros(E, device=dev)
+        k = max(top - 1, 1)
+        route = lambda: ops.moe_route(h, wr, None, k, scoring=ops.ROUTE_SIGMOID_PLAIN)          # noqa: E731
+        ms = _time(route, flush)
+        line("moe_route (sigmoid scores as they are)", phase, ms, bytes_=rows * D * 2 + E * D * 2, flops=2 * rows * E * D, like="moe_route (Tonilix)")
+        ms = _time(lambda: ops.moe_route(h, wr, rb, k, ops.ROUTE_SIGMOID_GROUPED, 8, 4, 2.0), flush)
+        line("moe_route (Tonilix: 4 of 8 groups)", phase, ms, bytes_=rows * D * 2 + E * D * 2, flops=2 * rows * E * D)
+        ids, wts = route()
+        wgu, wd = (torch.randn(E, 2 * F, D, device=dev) * D ** -0.5).to(bf), (torch.randn(E, D, F, device=dev) * F ** -0.5).to(bf)
+        path = "vendor grouped GEMM" if rows * k >= ops.MOE_GROUPED_GEMM_MIN_PAIRS else "own tiled kernels"
+        work = dict(bytes_=int(ids.unique().numel()) * 3 * F * D * 2, flops=6 * rows * k * F * D)
+        ms = _time(lambda: ops.moe_experts(h, ids, wts, wgu[:, :F], wgu[:, F:], wd, w_gate_up=wgu, weight_on_input=True, add=y), flush)
+        line(f"moe_experts (weights on the input, shared rows added; {path})", phase, ms, like="moe_experts (Kofadra)", **work)
+        ms = _time(lambda: ops.moe_experts(h, ids, wts, wgu[:, :F], wgu[:, F:], wd, w_gate_up=wgu), flush)
+        line(f"moe_experts (Kofadra; {path})", phase, ms, **work)
+        del wgu, wd, gu
+        torch.cuda.empty_cache()
+
+
 def run(family: str, sizes, steps: int, kernels: bool = True) -> None:
     import torch
     from b200attn.model import ModelConfig
-    if family not in ("kofadra", "gatolix", "tonilix", "sanarax", "gapidra"):
+    if family not in ("kofadra", "gatolix", "tonilix", "sanarax", "gapidra", "lizazen"):
         raise SystemExit(f"unknown family {family!r}")
     B, ctx, T = 64, 2560, 4096          # ctx: 2.5 mask blocks / windows of the bench geometries
     for name in sizes:
@@ -772,6 +918,11 @@ def run(family: str, sizes, steps: int, kernels: bool = True) -> None:
             s = GAPIDRA_SIZES[name]
             fcfg = bench_config(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["head_dim"], s["ff"], s["vocab"],
                                 kv_rank=s["kv_rank"], rot_dim=s["rot_dim"], window=s["window"], name=f"gapidra-{name}")
+        elif family == "lizazen":
+            from b200attn.lizazen import bench_config
+            s = LIZAZEN_SIZES[name]
+            fcfg = bench_config(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["head_dim"], s["ff"], s["experts"], s["top"],
+                                s["vocab"], window=s["window"], keep_first=s["keep_first"], chunk=s["chunk"], name=f"lizazen-{name}")
         else:
             from b200attn.gatolix import bench_config
             s = GATOLIX_SIZES[name]
@@ -800,8 +951,13 @@ def run(family: str, sizes, steps: int, kernels: bool = True) -> None:
                                   kv_rank=g["kv_rank"], q_rank=g["q_rank"], rot_dim=g["rot_dim"], window=g["window"],
                                   keep_first=g["keep_first"], name=f"sanarax-{name}")
             _throughput(scfg.name, scfg, B, ctx, T, steps)
+        if family == "lizazen":                 # the closest family at equal size: a parallel mixer, routed experts
+            from b200attn.tonilix import bench_config as tonilix_config
+            tcfg = tonilix_config(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["head_dim"], s["ff"], s["experts"], s["top"],
+                                  s["vocab"], name=f"tonilix-{name}")
+            _throughput(tcfg.name, tcfg, B, ctx, T, steps)
         _throughput(lcfg.name, lcfg, B, ctx, T, steps)
         if kernels:
             {"kofadra": _kernels_kofadra, "gatolix": _kernels_gatolix, "tonilix": _kernels_tonilix,
-             "sanarax": _kernels_sanarax, "gapidra": _kernels_gapidra}[family](name, s, B, ctx, T)
+             "sanarax": _kernels_sanarax, "gapidra": _kernels_gapidra, "lizazen": _kernels_lizazen}[family](name, s, B, ctx, T)
         torch.cuda.empty_cache()
