@@ -38,8 +38,8 @@ _oracle_cache = {}
 def _oracle(cfg, W, toks):
     key = (id(W), tuple(toks))
     if key not in _oracle_cache:
-        _oracle_cache[key] = U.oracle_logits(cfg, W, toks)
-    return _oracle_cache[key]
+        _oracle_cache[key] = W, U.oracle_logits(cfg, W, toks)      # W stays alive: its id names the entry
+    return _oracle_cache[key][1]
 
 
 def _check(got, cfg, W, reqs, dtype, what=""):

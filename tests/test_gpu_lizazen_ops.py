@@ -505,7 +505,7 @@ def test_experts_weighted_on_their_input(cuda, dt, T, E, top, D, F, glu, shared)
 
 @pytest.mark.parametrize("dt", DTYPES)
 @pytest.mark.parametrize("limit", [0.3, 1.0, 7.0])
-@pytest.mark.parametrize("ff", [22, 320])
+@pytest.mark.parametrize("ff", [22, 324])
 def test_bounded_units(cuda, dt, limit, ff):
     from b200attn.lizazen import GLU_ALPHA
     ops = _ops()
